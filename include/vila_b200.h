@@ -70,7 +70,9 @@ int vila_device_info(int* sm_count, int* cc_major, int* cc_minor);
 int vila_linear(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* bias,
                 const void* residual, int64_t ld_res, int res_row_mod, void* out, int64_t ldo,
                 int M, int N, int K, int act, int flags, void* stream);
-/* vila_linear with the coefficients of a two-parameter activation (VILA_ACT_XIELU: act_pos, act_neg); no residual. */
+/* vila_linear with the coefficients of a two-parameter activation (VILA_ACT_XIELU: act_pos, act_neg), or, with
+ * VILA_FLAG_GLU_CLAMP in flags, the clamped gated unit over interleaved weight rows (alpha = act_pos, limit =
+ * act_neg; out is [M, N / 2], N a multiple of 32, act none); no residual. */
 int vila_linear_act(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* bias, void* out, int64_t ldo,
                     int M, int N, int K, int act, float act_pos, float act_neg, int flags, void* stream);
 /* test hook: same, forcing the kernel configuration instead of the size heuristic:
@@ -538,6 +540,12 @@ typedef struct vila_rope_append_params {
   int32_t v_from_k;
   int32_t rot_layout; /* 0: pairs (2i, 2i+1); 1: pairs (i, i + rot_dims / 2) */
   float rot_mscale;   /* cos and sin are multiplied by this; 0 counts as 1 */
+  /* v_first != NULL: the cached value is (1 - v_mix) v + v_mix v_first[t, :] (G * vdim columns: another layer's values of the
+   * same tokens); not with v_from_k */
+  const void* v_first;
+  int64_t ld_vf;
+  int32_t v_first_dtype;
+  float v_mix;
 } vila_rope_append_params;
 int vila_rope_append(const vila_rope_append_params* p, void* stream);
 
@@ -577,6 +585,9 @@ typedef struct vila_paged_attn_params {
    * head_scale fp32 [H] or NULL: the scores of head h are multiplied by head_scale[h] (before mixing). */
   int32_t window, keep_first, talk_after;
   const float* head_scale;
+  /* softcap > 0: every head's own score becomes softcap * tanh(score / softcap), after scale and head_scale and
+   * before mixing, bias and softmax; 0: off */
+  float softcap;
 } vila_paged_attn_params;
 int vila_paged_attention(const vila_paged_attn_params* p, void* stream);
 
@@ -669,6 +680,8 @@ typedef struct vila_causal_conv_params {
 } vila_causal_conv_params;
 int vila_causal_conv_rows(const vila_causal_conv_params* p, void* stream);
 int vila_causal_conv_state(const vila_causal_conv_params* p, void* stream);
+/* Convolution and tail update in one launch for a step in which every sequence brings ONE row (rows == nseq). */
+int vila_causal_conv_step(const vila_causal_conv_params* p, void* stream);
 
 /* vila_ssd_scan — recurrence with one decay per head (state-space duality form), fp32 state:
  *   dt_t = softplus(dt_raw_t + dt_bias_h),  S_t = exp(-exp(A_log_h) dt_t) S_{t-1} + dt_t B_t x_t^T,
@@ -716,6 +729,61 @@ typedef struct vila_selective_scan_params {
   int32_t in_dtype, out_dtype, nseq, C, N;
 } vila_selective_scan_params;
 int vila_selective_scan(const vila_selective_scan_params* p, void* stream);
+
+/* ---- Outer-product recurrences with an fp32 state [slots, H, vdim, dim] (dim fastest), seqs as above; a
+ * sequence at position 0 starts from zero.  All arithmetic fp32 whatever the inputs' dtype. ------------- */
+
+/* vila_delta_scan — gated delta rule, per head h (q / k head h / (H / G)):
+ *   k^ = k / sqrt(sum k^2 + unit_eps),  q^ = q_scale q / sqrt(sum q^2 + unit_eps)
+ *   g = exp(-exp(A_log_h) softplus(a_t,h + dt_bias_h)),  beta = sigmoid(b_t,h)
+ *   S <- g S;  u = beta (v - S^T k^);  S <- S + k^ u^T;  out = S^T q^
+ * qkv rows hold q (G heads of dim) | k (G heads of dim) | v (H heads of vdim).  out fp32 [rows, ld_out]. */
+typedef struct vila_delta_scan_params {
+  const void* qkv;
+  int64_t ld_qkv;
+  const void* a; /* [rows, ld_a], column h */
+  int64_t ld_a;
+  const void* b; /* [rows, ld_b], column h */
+  int64_t ld_b;
+  const float* A_log;   /* [H] */
+  const float* dt_bias; /* [H] */
+  float* state;
+  const int32_t* seqs;
+  float* out;
+  int64_t ld_out;
+  int32_t in_dtype, ab_dtype, nseq, H, G, dim, vdim;
+  float q_scale, unit_eps;
+} vila_delta_scan_params;
+int vila_delta_scan(const vila_delta_scan_params* p, void* stream);
+
+/* vila_gla_scan — gated linear attention with one decay per key channel, per head:
+ *   alpha = sigmoid(z + z_bias)^(1 / tau);  S <- diag(alpha) S + k v^T;  out = S^T (q_scale q)
+ * q, k, z rows hold H heads of dim, v rows H heads of vdim.  out fp32 [rows, ld_out]. */
+typedef struct vila_gla_scan_params {
+  const void *q, *k, *v;
+  int64_t ld_q, ld_k, ld_v;
+  const void* z;
+  int64_t ld_z;
+  const float* z_bias; /* [H * dim] or NULL */
+  float* state;
+  const int32_t* seqs;
+  float* out;
+  int64_t ld_out;
+  int32_t in_dtype, z_dtype, nseq, H, dim, vdim;
+  float q_scale, tau;
+} vila_gla_scan_params;
+int vila_gla_scan(const vila_gla_scan_params* p, void* stream);
+
+/* Read-out of a recurrent mixer: out[t, h, :] = rms(o[t, h, :]) * w * silu(gate[t, h, :]), rms(v) = v / sqrt(mean(v^2)
+ * + eps) over the head's vdim columns, w [vdim] shared by the heads.  o and out are [rows, H * vdim] contiguous. */
+int vila_gated_head_norm_rows(const float* o, const float* w, const void* gate, int gate_dtype, int64_t ldg, float eps,
+                              void* out, int out_dtype, int rows, int H, int vdim, void* stream);
+
+/* Parallel-sublayer residual in one pass: x[r, :] += a_scale * a[r, :] + b_scale * b[r, :] (per-channel fp32 scales; b may
+ * be NULL), then, if out != NULL, out[r, :] = x[r, :] / sqrt(mean(x[r, :]^2) + eps) * w (w fp32 or NULL). */
+int vila_scaled_residual_norm_rows(float* x, const void* a, int a_dtype, int64_t lda, const float* a_scale, const void* b,
+                                   int b_dtype, int64_t ldb, const float* b_scale, const float* w, float eps, void* out,
+                                   int out_dtype, int rows, int cols, void* stream);
 
 #ifdef __cplusplus
 }

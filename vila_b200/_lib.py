@@ -136,6 +136,7 @@ class RopeAppendParams(C.Structure):
         ("unit_norm", C.c_int32), ("eps", c_float),
         ("q_norm_w", c_void_p), ("k_norm_w", c_void_p), ("v_from_k", C.c_int32),
         ("rot_layout", C.c_int32), ("rot_mscale", c_float),
+        ("v_first", c_void_p), ("ld_vf", c_i64), ("v_first_dtype", C.c_int32), ("v_mix", c_float),
     ]
 
 
@@ -149,6 +150,7 @@ class PagedAttnParams(C.Structure):
         ("dist_bias", c_void_p), ("gate", c_void_p), ("ldg", c_i64),
         ("dist_rows", C.c_int32), ("chunk", C.c_int32), ("gate_dtype", C.c_int32),
         ("window", C.c_int32), ("keep_first", C.c_int32), ("talk_after", C.c_int32), ("head_scale", c_void_p),
+        ("softcap", c_float),
     ]
 
 
@@ -177,6 +179,26 @@ class SelectiveScanParams(C.Structure):
         ("z", c_void_p), ("ld_z", c_i64), ("dt_bias", c_void_p), ("A_log", c_void_p), ("D", c_void_p),
         ("state", c_void_p), ("seqs", c_void_p), ("out", c_void_p), ("ld_out", c_i64),
         ("in_dtype", C.c_int32), ("out_dtype", C.c_int32), ("nseq", C.c_int32), ("C", C.c_int32), ("N", C.c_int32),
+    ]
+
+
+class DeltaScanParams(C.Structure):
+    _fields_ = [
+        ("qkv", c_void_p), ("ld_qkv", c_i64), ("a", c_void_p), ("ld_a", c_i64), ("b", c_void_p), ("ld_b", c_i64),
+        ("A_log", c_void_p), ("dt_bias", c_void_p), ("state", c_void_p), ("seqs", c_void_p), ("out", c_void_p),
+        ("ld_out", c_i64),
+        ("in_dtype", C.c_int32), ("ab_dtype", C.c_int32), ("nseq", C.c_int32), ("H", C.c_int32), ("G", C.c_int32),
+        ("dim", C.c_int32), ("vdim", C.c_int32), ("q_scale", c_float), ("unit_eps", c_float),
+    ]
+
+
+class GlaScanParams(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("ld_q", c_i64), ("ld_k", c_i64), ("ld_v", c_i64),
+        ("z", c_void_p), ("ld_z", c_i64), ("z_bias", c_void_p), ("state", c_void_p), ("seqs", c_void_p),
+        ("out", c_void_p), ("ld_out", c_i64),
+        ("in_dtype", C.c_int32), ("z_dtype", C.c_int32), ("nseq", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32),
+        ("vdim", C.c_int32), ("q_scale", c_float), ("tau", c_float),
     ]
 
 
@@ -271,7 +293,14 @@ SIGNATURES = {
                                   c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "vila_causal_conv_rows": [C.POINTER(CausalConvParams), c_void_p],
     "vila_causal_conv_state": [C.POINTER(CausalConvParams), c_void_p],
+    "vila_causal_conv_step": [C.POINTER(CausalConvParams), c_void_p],
     "vila_ssd_scan": [C.POINTER(SsdScanParams), c_void_p],
+    "vila_delta_scan": [C.POINTER(DeltaScanParams), c_void_p],
+    "vila_gla_scan": [C.POINTER(GlaScanParams), c_void_p],
+    "vila_gated_head_norm_rows": [c_void_p, c_void_p, c_void_p, c_int, c_i64, c_float, c_void_p, c_int, c_int, c_int,
+                                  c_int, c_void_p],
+    "vila_scaled_residual_norm_rows": [c_void_p, c_void_p, c_int, c_i64, c_void_p, c_void_p, c_int, c_i64, c_void_p,
+                                       c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     "vila_selective_scan": [C.POINTER(SelectiveScanParams), c_void_p],
 }
 _RESTYPES = {"vila_last_error": C.c_char_p}

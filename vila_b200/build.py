@@ -37,6 +37,7 @@ SOURCES = [
     "short_conv.cu",
     "paged_attn.cu",
     "ssm.cu",
+    "outer_scan.cu",
 ]
 HEADERS = ["common.cuh", "kernels.h", "dtype_any.cuh", "../../include/vila_b200.h"]
 

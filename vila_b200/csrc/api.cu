@@ -82,6 +82,10 @@ int vila_linear_act(const void* x, int64_t ldx, const void* w, int64_t ldw, cons
   vb::GemmEpilogue e = make_epi(bias, nullptr, 0, 0, act, flags);
   e.act_pos = act_pos;
   e.act_neg = act_neg;
+  if (flags & VILA_FLAG_GLU_CLAMP) {
+    VB_CHECK(act == VILA_ACT_NONE, "vila_linear_act: the clamped gated unit takes no other activation (act=%d)", act);
+    e.swiglu = 2;
+  }
   return vb::gemm_bf16(cb(x), (int)ldx, cb(w), (int)ldw, mb(out), (int)ldo, M, N, K, e, st(stream));
 }
 
@@ -520,6 +524,35 @@ int vila_causal_conv_rows(const vila_causal_conv_params* p, void* stream) {
 int vila_causal_conv_state(const vila_causal_conv_params* p, void* stream) {
   VB_REQUIRE_DEVICE();
   return vb::causal_conv_state(*p, st(stream));
+}
+
+int vila_causal_conv_step(const vila_causal_conv_params* p, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::causal_conv_step(*p, st(stream));
+}
+
+int vila_delta_scan(const vila_delta_scan_params* p, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::delta_scan(*p, st(stream));
+}
+
+int vila_gla_scan(const vila_gla_scan_params* p, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::gla_scan(*p, st(stream));
+}
+
+int vila_scaled_residual_norm_rows(float* x, const void* a, int a_dtype, int64_t lda, const float* a_scale, const void* b,
+                                   int b_dtype, int64_t ldb, const float* b_scale, const float* w, float eps, void* out,
+                                   int out_dtype, int rows, int cols, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::scaled_residual_norm_rows(x, a, a_dtype, lda, a_scale, b, b_dtype, ldb, b_scale, w, eps, out, out_dtype, rows,
+                                       cols, st(stream));
+}
+
+int vila_gated_head_norm_rows(const float* o, const float* w, const void* gate, int gate_dtype, int64_t ldg, float eps,
+                              void* out, int out_dtype, int rows, int H, int vdim, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::gated_head_norm_rows(o, w, gate, gate_dtype, ldg, eps, out, out_dtype, rows, H, vdim, st(stream));
 }
 
 int vila_ssd_scan(const vila_ssd_scan_params* p, void* stream) {

@@ -87,6 +87,11 @@ __device__ __forceinline__ float xielu_fast_f(float z, float a_pos, float a_neg)
   const float neg = a_neg * (__expf(zn) - 1.0f - zn), pos = a_pos * z * z;
   return fmaf(0.5f, z, z > 0.f ? pos : neg);
 }
+// clamped gated unit: g = min(zg, limit), u = clamp(zu, +-limit): g sigmoid(alpha g) (u + 1)
+__device__ __forceinline__ float glu_clamp_fast_f(float zg, float zu, float alpha, float limit) {
+  const float g = fminf(zg, limit), u = fminf(fmaxf(zu, -limit), limit);
+  return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
 __device__ __forceinline__ float gelu_erf_f(float x) {
   return 0.5f * x * (1.0f + erff(x * 0.7071067811865476f));
 }

@@ -16,6 +16,8 @@
 // query and key (dist_bias [dist_rows, H], the last row serves every larger distance; added after scale and
 // mixing), a chunked mask (a query sees the keys of its own block of `chunk` positions only; the key loop
 // starts at the block of the tile's first row), and a per-(token, head) sigmoid gate on the output.
+// A cap bounds every head's own scaled score to softcap * tanh(score / softcap) before mixing, bias and softmax.
+// The append kernel can mix another layer's values of the same tokens into the cached ones.
 // A sliding window with kept first tokens (a key is seen if it is at most window - 1 positions back, or among the
 // first keep_first of its sequence) is a mask plus a shorter block list: the blocks that hold kept tokens, then
 // the blocks from the window of the tile's first row on.  A per-head multiplier of the scores is folded into the
@@ -100,8 +102,12 @@ __global__ void __launch_bounds__(kThreads) rope_append_kernel(const vila_rope_a
   }
   if (p.v_from_k) return;
   const size_t vsrc = in0 + static_cast<size_t>(p.H + p.G) * p.dim, vdst = prow + static_cast<size_t>(p.G) * p.dim;
-  for (int c = tid; c < p.G * p.vdim; c += kThreads)
-    st_any(p.pool, p.pool_dtype, vdst + c, ld_any(p.qkv, p.qkv_dtype, vsrc + c));
+  for (int c = tid; c < p.G * p.vdim; c += kThreads) {
+    float v = ld_any(p.qkv, p.qkv_dtype, vsrc + c);
+    if (p.v_first)   // part of the value comes from another layer's value of the same token
+      v = fmaf(p.v_mix, ld_any(p.v_first, p.v_first_dtype, static_cast<size_t>(t) * p.ld_vf + c), (1.0f - p.v_mix) * v);
+    st_any(p.pool, p.pool_dtype, vdst + c, v);
+  }
 }
 
 // ---- attention -----------------------------------------------------------------------------------------
@@ -148,6 +154,10 @@ __device__ __forceinline__ BlockList visible_blocks(const vila_paged_attn_params
 }
 __device__ __forceinline__ float head_scale(const vila_paged_attn_params& p, int h) {
   return p.head_scale ? p.scale * p.head_scale[h] : p.scale;
+}
+// a head's own scaled score, bounded to (-softcap, softcap) when a cap is set
+__device__ __forceinline__ float capped(const vila_paged_attn_params& p, float s) {
+  return p.softcap > 0.f ? p.softcap * tanhf(s / p.softcap) : s;
 }
 __device__ __forceinline__ float dist_bias(const vila_paged_attn_params& p, int dist, int h) {
   return __ldg(p.dist_bias + static_cast<size_t>(min(dist, p.dist_rows - 1)) * p.H + h);
@@ -307,7 +317,7 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
         const float4 a = qr[k], c = kr[k];
         s = fmaf(a.x, c.x, s); s = fmaf(a.y, c.y, s); s = fmaf(a.z, c.z, s); s = fmaf(a.w, c.w, s);
       }
-      Ss[idx] = s;
+      Ss[idx] = capped(p, s);
     }
     __syncthreads();
     if (after) {
@@ -351,9 +361,13 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
       const bool valid = lane < BK && i < n && sees(p, pos0 + i, j0 + lane);
       float s = 0.f;
       if (lane < BK) {
-        const float* tk = Tk + h * H;
-        const float* sr = Ss + (i * H) * BK + lane;
-        for (int g = 0; g < H; ++g) s = fmaf(tk[g], sr[g * BK], s);
+        if (p.talk) {
+          const float* tk = Tk + h * H;
+          const float* sr = Ss + (i * H) * BK + lane;
+          for (int g = 0; g < H; ++g) s = fmaf(tk[g], sr[g * BK], s);
+        } else {
+          s = Ss[r * BK + lane];
+        }
       }
       if (valid && p.dist_bias) s += dist_bias(p, pos0 + i - (j0 + lane), h);
       s = valid ? s : kNegBig;
@@ -507,8 +521,8 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
       }
 #pragma unroll
       for (int a = 0; a < TR; ++a) {
-        Ss[(r0 + a) * BK + jp] = s[a][0];
-        Ss[(r0 + a) * BK + jp + HK] = s[a][1];
+        Ss[(r0 + a) * BK + jp] = capped(p, s[a][0]);
+        Ss[(r0 + a) * BK + jp + HK] = capped(p, s[a][1]);
       }
     }
     __syncthreads();
@@ -560,15 +574,19 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
           const int h = r / BQ, i = r - h * BQ;
           ok[u] = lane < BK && i < n && sees(p, pos0 + i, j0 + lane);
           if (lane < BK) {
-            const float* tk = Tk + h * H;
-            const float* sr = Ss + i * BK + lane;
             float s0 = 0.f, s1 = 0.f;
-            int g = 0;
-            for (; g + 1 < H; g += 2) {
-              s0 = fmaf(tk[g], sr[g * BQ * BK], s0);
-              s1 = fmaf(tk[g + 1], sr[(g + 1) * BQ * BK], s1);
+            if (p.talk) {
+              const float* tk = Tk + h * H;
+              const float* sr = Ss + i * BK + lane;
+              int g = 0;
+              for (; g + 1 < H; g += 2) {
+                s0 = fmaf(tk[g], sr[g * BQ * BK], s0);
+                s1 = fmaf(tk[g + 1], sr[(g + 1) * BQ * BK], s1);
+              }
+              if (g < H) s0 = fmaf(tk[g], sr[g * BQ * BK], s0);
+            } else {
+              s0 = Ss[r * BK + lane];
             }
-            if (g < H) s0 = fmaf(tk[g], sr[g * BQ * BK], s0);
             if (ok[u]) sv[u] = s0 + s1 + (p.dist_bias ? dist_bias(p, pos0 + i - (j0 + lane), h0 + h) : 0.f);
           }
           mo[u] = m_s[r];
@@ -709,6 +727,7 @@ int paged_attention(const vila_paged_attn_params& p, cudaStream_t stream) {
   constexpr size_t kSmemMax = 224 * 1024;
   VB_CHECK(p.chunk >= 0 && (p.dist_bias == nullptr || p.dist_rows >= 1), "paged_attention: chunk=%d dist_rows=%d",
            p.chunk, p.dist_rows);
+  VB_CHECK(p.softcap >= 0.f, "paged_attention: softcap=%f", p.softcap);
   VB_CHECK(p.window >= 0 && p.keep_first >= 0 && (p.talk_after == 0 || (p.talk != nullptr && p.sink == nullptr)),
            "paged_attention: window=%d keep_first=%d; talk_after needs talk and no sink", p.window, p.keep_first);
   VB_CHECK(p.max_rows >= 1 && p.max_rows <= 16 && (p.nsplit == 1 || p.max_rows == 1),

@@ -441,7 +441,182 @@ branch_norm_residual_kernel(float* __restrict__ x, const void* __restrict__ a, i
   }
 }
 
+// ---- parallel-sublayer residual with per-channel scales ------------------------------------------------
+// x += sa * a + sb * b (element by element; sa / sb one vector each, b may be missing), then, if out is given,
+// out = x / sqrt(mean(x^2) + eps) * w: the operand of both sublayers of the next layer.  The vector form keeps
+// the row in registers between the sum and the norm.
+struct ScaledResidual {
+  float* x;
+  const void *a, *b;
+  int64_t lda, ldb;
+  const float *sa, *sb, *w;
+  void* out;
+  int a_dt, b_dt, o_dt, rows, cols;
+  float eps;
+};
+
+__device__ __forceinline__ float4 ld4_any(const void* p, int dt, size_t i) {
+  if (dt) return *reinterpret_cast<const float4*>(static_cast<const float*>(p) + i);
+  const uint2 u = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p) + i);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                     __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void st4_any(void* p, int dt, size_t i, float4 v) {
+  if (dt) {
+    *reinterpret_cast<float4*>(static_cast<float*>(p) + i) = v;
+    return;
+  }
+  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<unsigned int*>(&lo);
+  u.y = *reinterpret_cast<unsigned int*>(&hi);
+  *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p) + i) = u;
+}
+
+template <int TPR>
+__global__ void __launch_bounds__(kRowThreads) scaled_residual_norm_kernel(const ScaledResidual p) {
+  __shared__ float red[kRowsPerCta];
+  const int row = row_of<TPR>();
+  if (row >= p.rows) return;
+  float* xr = p.x + static_cast<size_t>(row) * p.cols;
+  const size_t ab = static_cast<size_t>(row) * p.lda, bb = static_cast<size_t>(row) * p.ldb;
+  float ss = 0.f;
+  for (int c = col0_of<TPR>(); c < p.cols; c += TPR) {
+    float y = p.sa[c] * ld_any(p.a, p.a_dt, ab + c);
+    if (p.b) y = fmaf(p.sb[c], ld_any(p.b, p.b_dt, bb + c), y);
+    const float v = xr[c] + y;
+    xr[c] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (!p.out) return;
+  ss = row_sum<TPR>(ss, red);
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(p.cols) + p.eps);
+  for (int c = col0_of<TPR>(); c < p.cols; c += TPR)
+    st_any(p.out, p.o_dt, static_cast<size_t>(row) * p.cols + c, xr[c] * r * (p.w ? p.w[c] : 1.0f));
+}
+
+template <int TPR, int NV>   // cols <= 4 * TPR * NV, a multiple of 4, all rows aligned
+__global__ void __launch_bounds__(kRowThreads) scaled_residual_norm_vec_kernel(const ScaledResidual p) {
+  __shared__ float red[kRowsPerCta];
+  const int row = row_of<TPR>();
+  if (row >= p.rows) return;
+  float* xr = p.x + static_cast<size_t>(row) * p.cols;
+  const size_t ab = static_cast<size_t>(row) * p.lda, bb = static_cast<size_t>(row) * p.ldb;
+  float4 v[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = 4 * (col0_of<TPR>() + TPR * k);
+    v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < p.cols) {
+      const float4 x4 = *reinterpret_cast<const float4*>(xr + c), a4 = ld4_any(p.a, p.a_dt, ab + c);
+      const float4 s4 = __ldg(reinterpret_cast<const float4*>(p.sa + c));
+      float4 y = make_float4(s4.x * a4.x, s4.y * a4.y, s4.z * a4.z, s4.w * a4.w);
+      if (p.b) {
+        const float4 b4 = ld4_any(p.b, p.b_dt, bb + c), t4 = __ldg(reinterpret_cast<const float4*>(p.sb + c));
+        y.x = fmaf(t4.x, b4.x, y.x); y.y = fmaf(t4.y, b4.y, y.y); y.z = fmaf(t4.z, b4.z, y.z); y.w = fmaf(t4.w, b4.w, y.w);
+      }
+      v[k] = make_float4(x4.x + y.x, x4.y + y.y, x4.z + y.z, x4.w + y.w);
+      *reinterpret_cast<float4*>(xr + c) = v[k];
+    }
+    ss = fmaf(v[k].x, v[k].x, ss); ss = fmaf(v[k].y, v[k].y, ss);
+    ss = fmaf(v[k].z, v[k].z, ss); ss = fmaf(v[k].w, v[k].w, ss);
+  }
+  if (!p.out) return;
+  ss = row_sum<TPR>(ss, red);
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(p.cols) + p.eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = 4 * (col0_of<TPR>() + TPR * k);
+    if (c < p.cols) {
+      float4 w4 = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (p.w) w4 = __ldg(reinterpret_cast<const float4*>(p.w + c));
+      st4_any(p.out, p.o_dt, static_cast<size_t>(row) * p.cols + c,
+              make_float4(v[k].x * r * w4.x, v[k].y * r * w4.y, v[k].z * r * w4.z, v[k].w * r * w4.w));
+    }
+  }
+}
+
+// ---- read-out of a recurrent mixer: per-head RMS norm, shared weight, SiLU gate ---------------------------
+// out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * w * silu(gate[t, h, :]); a warp per (token, head)
+template <bool VEC>
+__global__ void __launch_bounds__(kRowThreads)
+gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, const void* __restrict__ gate, int g_dt,
+                       int64_t ldg, float eps, void* __restrict__ out, int o_dt, int pairs, int H, int vdim) {
+  const int pair = blockIdx.x * kRowsPerCta + (threadIdx.x >> 5);
+  if (pair >= pairs) return;
+  const int t = pair / H, h = pair - t * H, lane = threadIdx.x & 31;
+  const size_t ob = static_cast<size_t>(pair) * vdim, gb = static_cast<size_t>(t) * ldg + static_cast<size_t>(h) * vdim;
+  float ss = 0.f;
+  if (VEC) {
+    for (int c = 4 * lane; c < vdim; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(o + ob + c);
+      ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+    }
+  } else {
+    for (int c = lane; c < vdim; c += 32) ss = fmaf(o[ob + c], o[ob + c], ss);
+  }
+  ss = warp_sum(ss);
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(vdim) + eps);
+  if (VEC) {
+    for (int c = 4 * lane; c < vdim; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(o + ob + c), g = ld4_any(gate, g_dt, gb + c);
+      const float4 w4 = __ldg(reinterpret_cast<const float4*>(w + c));
+      st4_any(out, o_dt, ob + c, make_float4(v.x * r * w4.x * silu_exact_f(g.x), v.y * r * w4.y * silu_exact_f(g.y),
+                                             v.z * r * w4.z * silu_exact_f(g.z), v.w * r * w4.w * silu_exact_f(g.w)));
+    }
+  } else {
+    for (int c = lane; c < vdim; c += 32)
+      st_any(out, o_dt, ob + c, o[ob + c] * r * w[c] * silu_exact_f(ld_any(gate, g_dt, gb + c)));
+  }
+}
+
+inline bool aligned_to(const void* p, size_t n) { return reinterpret_cast<uintptr_t>(p) % n == 0; }
+// rows of a [.., ld] tensor that start on a four-element boundary (8 bytes bf16, 16 bytes fp32)
+inline bool rows4(const void* p, int64_t ld, int dt) { return ld % 4 == 0 && aligned_to(p, dt ? 16 : 8); }
+
 }  // namespace
+
+int scaled_residual_norm_rows(float* x, const void* a, int a_dt, int64_t lda, const float* sa, const void* b, int b_dt,
+                              int64_t ldb, const float* sb, const float* w, float eps, void* out, int o_dt, int rows,
+                              int cols, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  VB_CHECK(cols > 0 && a != nullptr && sa != nullptr && (b == nullptr || sb != nullptr), "scaled_residual_norm_rows: cols=%d", cols);
+  const ScaledResidual p = {x, a, b, lda, ldb, sa, sb, w, out, a_dt, b_dt, o_dt, rows, cols, eps};
+  const bool vec = cols % 4 == 0 && aligned_to(x, 16) && aligned_to(sa, 16) && rows4(a, lda, a_dt) &&
+                   (b == nullptr || (rows4(b, ldb, b_dt) && aligned_to(sb, 16))) && (w == nullptr || aligned_to(w, 16)) &&
+                   (out == nullptr || aligned_to(out, o_dt ? 16 : 8));
+#define VB_SRN(K, G) VB_CUDA(launch_serial(K, dim3(G), dim3(kRowThreads), 0, stream, p))
+  if (cols >= kWideCols) {
+    if (vec && cols <= 1024) VB_SRN((scaled_residual_norm_vec_kernel<256, 1>), rows);
+    else if (vec && cols <= 2048) VB_SRN((scaled_residual_norm_vec_kernel<256, 2>), rows);
+    else if (vec && cols <= 4096) VB_SRN((scaled_residual_norm_vec_kernel<256, 4>), rows);
+    else if (vec && cols <= 8192) VB_SRN((scaled_residual_norm_vec_kernel<256, 8>), rows);
+    else VB_SRN(scaled_residual_norm_kernel<256>, rows);
+  } else if (vec) {
+    VB_SRN((scaled_residual_norm_vec_kernel<32, 4>), row_grid(rows));
+  } else {
+    VB_SRN(scaled_residual_norm_kernel<32>, row_grid(rows));
+  }
+#undef VB_SRN
+  return 0;
+}
+
+int gated_head_norm_rows(const float* o, const float* w, const void* gate, int g_dt, int64_t ldg, float eps, void* out,
+                         int o_dt, int rows, int H, int vdim, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  VB_CHECK(H >= 1 && vdim >= 1 && w != nullptr && gate != nullptr, "gated_head_norm_rows: H=%d vdim=%d", H, vdim);
+  VB_CHECK(static_cast<long>(rows) * H < (1L << 31), "gated_head_norm_rows: rows=%d H=%d", rows, H);
+  const int pairs = rows * H;
+  const bool vec = vdim % 4 == 0 && aligned_to(o, 16) && aligned_to(w, 16) && rows4(gate, ldg, g_dt) && aligned_to(out, o_dt ? 16 : 8);
+  if (vec)
+    VB_CUDA(launch_serial(gated_head_norm_kernel<true>, dim3(row_grid(pairs)), dim3(kRowThreads), 0, stream, o, w, gate, g_dt,
+                          ldg, eps, out, o_dt, pairs, H, vdim));
+  else
+    VB_CUDA(launch_serial(gated_head_norm_kernel<false>, dim3(row_grid(pairs)), dim3(kRowThreads), 0, stream, o, w, gate, g_dt,
+                          ldg, eps, out, o_dt, pairs, H, vdim));
+  return 0;
+}
 
 int embed_rows(const void* table, int dt, const int32_t* ids, float* out, int rows, int cols,
                cudaStream_t stream) {

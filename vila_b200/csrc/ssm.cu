@@ -8,6 +8,8 @@
 //                       registers (taps + rows - 1 loads for `rows` outputs); rows before the portion come
 //                       from the state [slots, taps - 1, cols], rows before position 0 are zero
 //   causal_conv_state   the last taps - 1 inputs of every sequence, after the convolution
+//   causal_conv_step    both in one launch when every sequence brings exactly one row (decoded tokens): the thread
+//                       that owns a channel reads the tail, writes the output and moves the tail up
 //   ssd_scan            S_t = a_t S_{t-1} + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t  with one decay
 //                       a_t = exp(-exp(A_log) dt_t) per head.  Grid (sequence, head, 32 columns of P);
 //                       thread (column c = tid / 8, r = tid % 8) keeps the state entries n = r * KPT .. of
@@ -103,6 +105,26 @@ __global__ void __launch_bounds__(kThreads) causal_conv_state_kernel(const vila_
       st[static_cast<size_t>(j) * p.cols + c] = v;
     }
   }
+}
+
+__global__ void __launch_bounds__(kThreads) causal_conv_step_kernel(const vila_causal_conv_params p) {
+  const int* sq = p.seqs + 4 * blockIdx.x;
+  const int row = sq[0], pos = sq[2], slot = sq[3], taps = p.taps, back = taps - 1;
+  const int c = blockIdx.y * kThreads + threadIdx.x;
+  if (c >= p.cols) return;
+  const float cur = ld_any(p.in, p.in_dtype, static_cast<size_t>(row) * p.ld_in + c);
+  float acc = p.bias ? ld_any(p.bias, p.w_dtype, c) : 0.f;
+  float* st = p.state + static_cast<size_t>(slot) * back * p.cols + c;
+  const size_t wb = static_cast<size_t>(c) * taps;
+  for (int j = 0; j < back; ++j) {   // tail row j holds the input back - j positions ago
+    const float v = pos - (back - j) >= 0 ? st[static_cast<size_t>(j) * p.cols] : 0.f;
+    acc = fmaf(ld_any(p.w, p.w_dtype, wb + j), v, acc);
+    if (j > 0) st[static_cast<size_t>(j - 1) * p.cols] = v;
+  }
+  acc = fmaf(ld_any(p.w, p.w_dtype, wb + back), cur, acc);
+  if (back > 0) st[static_cast<size_t>(back - 1) * p.cols] = cur;
+  if (p.act == VILA_CONV_SILU) acc = silu_exact_f(acc);
+  st_any(p.out, p.out_dtype, static_cast<size_t>(row) * p.ld_out + c, acc);
 }
 
 // ---- scalar-decay recurrence (state-space duality form) ----------------------------------------------
@@ -348,6 +370,16 @@ int causal_conv_rows(const vila_causal_conv_params& p, cudaStream_t stream) {
     default: VB_CONV(0); break;
   }
 #undef VB_CONV
+  return 0;
+}
+
+int causal_conv_step(const vila_causal_conv_params& p, cudaStream_t stream) {
+  if (p.rows <= 0 || p.cols <= 0) return 0;
+  VB_CHECK(p.rows == p.nseq && p.taps >= 1 && p.taps <= kMaxTaps && (p.taps == 1 || p.state != nullptr),
+           "causal_conv_step: rows=%d sequences=%d taps=%d", p.rows, p.nseq, p.taps);
+  const dim3 grid(p.nseq, (p.cols + kThreads - 1) / kThreads);
+  VB_CHECK(grid.y <= 65535, "causal_conv_step: cols=%d", p.cols);
+  VB_CUDA(launch_serial(causal_conv_step_kernel, grid, dim3(kThreads), 0, stream, p));
   return 0;
 }
 

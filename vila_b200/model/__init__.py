@@ -1,4 +1,5 @@
 """vila_b200.model — mirrors the names callers import from `llava.model`."""
+from .bivizen import BivizenConfig, BivizenForCausalLM, BivizenLayerConfig
 from .configuration import (LlavaConfig, Qwen2Config, SiglipVisionConfig, nvila_8b,
                             nvila_8b_dynamic_s2, nvila_lite_3b, nvila_video_8b, tiny_test_config)
 from .llava_llama import (BasicImageEncoder, BasicVideoEncoder, LlavaLlamaModel, SyntheticTokenizer,

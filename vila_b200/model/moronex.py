@@ -28,7 +28,7 @@ import json
 import struct
 from dataclasses import dataclass, field
 from pathlib import Path
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
@@ -168,6 +168,20 @@ def read_safetensors(path) -> Dict[str, torch.Tensor]:
     return out
 
 
+def stack_rows(parts: List[Tuple[str, torch.Tensor]]):
+    """Stack projections [out, in] that read the same input; every part starts at a multiple of 8 rows so
+    its output columns are 16-byte aligned views.  -> (weight, {name: (offset, rows)})"""
+    out, offs, at = [], {}, 0
+    for nm, t in parts:
+        offs[nm] = (at, t.shape[0])
+        pad = _pad8(t.shape[0]) - t.shape[0]
+        out.append(t)
+        if pad:
+            out.append(t.new_zeros(pad, t.shape[1]))
+        at += t.shape[0] + pad
+    return torch.cat(out, 0).contiguous(), offs
+
+
 class _Layer:
     """Device tensors of one layer in the layout the kernels want."""
 
@@ -239,18 +253,7 @@ class MoronexForCausalLM:
             return tensors[name].to(device=dev, dtype=torch.float32).contiguous()
 
         def cat_rows(names):
-            """Stack projections that read the same input; every part starts at a multiple of 8 rows so
-            its output columns are 16-byte aligned views.  -> (weight, {name: (offset, rows)})"""
-            parts, offs, at = [], {}, 0
-            for nm in names:
-                t = w(nm)
-                offs[nm] = (at, t.shape[0])
-                pad = _pad8(t.shape[0]) - t.shape[0]
-                parts.append(t)
-                if pad:
-                    parts.append(torch.zeros(pad, t.shape[1], device=dev, dtype=dt))
-                at += t.shape[0] + pad
-            return torch.cat(parts, 0).contiguous(), offs
+            return stack_rows([(nm, w(nm)) for nm in names])
 
         self.weights = {n: tensors[n] for n in want}
         self.embed, self.head, self.final_norm = w("embed"), w("head"), f32("final.norm")

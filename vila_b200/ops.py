@@ -49,16 +49,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
            act: int = ACT_NONE, residual: Optional[torch.Tensor] = None, res_row_mod: int = 0,
            swiglu: bool = False, out: Optional[torch.Tensor] = None,
            block_n: Optional[int] = None, static_w: bool = False,
-           act_params: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+           act_params: Optional[Tuple[float, float]] = None,
+           glu_clamp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """out = epilogue(x @ w.T).  x [M,K] (row stride arbitrary), w [N,K].
     static_w: w is a parameter (VILA_FLAG_STATIC_W): it may be fetched before the PDL wait.
-    act_params: the two coefficients of ACT_XIELU (positive side, negative side)."""
+    act_params: the two coefficients of ACT_XIELU (positive side, negative side).
+    glu_clamp = (alpha, limit): clamped gated unit over interleaved (gate, up) weight rows, see VILA_FLAG_GLU_CLAMP."""
     _chk(x, "x"); _chk(w, "w")
     assert x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1], (x.shape, w.shape)
     assert x.stride(1) == 1 and w.stride(1) == 1
     M, K = x.shape
     N = w.shape[0]
-    n_out = N // 2 if swiglu else N
+    n_out = N // 2 if (swiglu or glu_clamp is not None) else N
     if out is None:
         out = torch.empty((M, n_out), dtype=torch.bfloat16, device=x.device)
     else:
@@ -73,7 +75,12 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     lib = _lib.load()
     args = (_p(x), x.stride(0), _p(w), w.stride(0), _p(bias), _p(residual), ld_res, res_row_mod,
             _p(out), out.stride(0), M, N, K, act, (1 if swiglu else 0) | (2 if static_w else 0), _stream())
-    if act_params is not None:
+    if glu_clamp is not None:
+        assert residual is None and block_n is None and act == ACT_NONE and not swiglu
+        check(lib.vila_linear_act(_p(x), x.stride(0), _p(w), w.stride(0), _p(bias), _p(out), out.stride(0), M, N, K,
+                                  act, float(glu_clamp[0]), float(glu_clamp[1]), 4 | (2 if static_w else 0), _stream()),
+              "vila_linear_act")
+    elif act_params is not None:
         assert residual is None and block_n is None
         check(lib.vila_linear_act(_p(x), x.stride(0), _p(w), w.stride(0), _p(bias), _p(out), out.stride(0), M, N, K,
                                   act, float(act_params[0]), float(act_params[1]),
@@ -673,15 +680,16 @@ def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, tiles: tor
 # ---- parallel-sublayer decoders: pair embedding, short convolution, rotary GQA over a paged pool, sigmoid router ----
 def linear_any(x: torch.Tensor, w: torch.Tensor, *, swiglu: bool = False, out_dtype=None,
                bias: Optional[torch.Tensor] = None, act: int = ACT_NONE,
-               act_params: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+               act_params: Optional[Tuple[float, float]] = None,
+               glu_clamp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """act(x [M, K] · w[N, K]^T + bias): bf16 operands with 16-byte aligned rows go to the tcgen05 GEMM,
     everything else (fp32 tensors, odd shapes, an fp32 result) to the CUDA-core grouped kernel."""
     N, K = w.shape
     if (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and out_dtype in (None, torch.bfloat16)
             and K % 8 == 0 and N % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
-            and (not swiglu or N % 32 == 0)):
-        return linear(x, w, bias, act=act, swiglu=swiglu, static_w=True, act_params=act_params)
-    return glinear(x, w, swiglu=swiglu, out_dtype=out_dtype, bias=bias, act=act, act_params=act_params)
+            and (not (swiglu or glu_clamp) or N % 32 == 0)):
+        return linear(x, w, bias, act=act, swiglu=swiglu, static_w=True, act_params=act_params, glu_clamp=glu_clamp)
+    return glinear(x, w, swiglu=swiglu, out_dtype=out_dtype, bias=bias, act=act, act_params=act_params, glu_clamp=glu_clamp)
 
 
 def embed_pair_rows(table: torch.Tensor, pair_table: torch.Tensor, ids: torch.Tensor, prev_ids: torch.Tensor,
@@ -760,13 +768,14 @@ def rope_append(qkv: torch.Tensor, positions: torch.Tensor, cache_rows: torch.Te
                 heads: int, kv_heads: int, dim: int, vdim: int, inv_freq: Optional[torch.Tensor],
                 unit_norm: bool, eps: float, q_norm_w: Optional[torch.Tensor] = None,
                 k_norm_w: Optional[torch.Tensor] = None, v_from_k: bool = False, halves: bool = False,
-                mscale: float = 1.0) -> torch.Tensor:
+                mscale: float = 1.0, v_first: Optional[torch.Tensor] = None, v_mix: float = 0.0) -> torch.Tensor:
     """qkv [T, >= heads*dim + kv_heads*(dim+vdim)] -> q fp32 [T, heads*dim] (rotated, unit-normed); the
     token's k | v go to row cache_rows[t] of pool [pool rows, kv_heads*(dim+vdim)].  inv_freq float64
     [rot_dims / 2] (None: no rotation).  q_norm_w / k_norm_w fp32 [dim]: weights of the per-head norm.
     v_from_k: qkv holds q | k only, the cached value of a token is its incoming key (before rotation / norm).
     halves: column i of the rotated part pairs with i + rot_dims / 2 instead of 2i with 2i + 1; mscale multiplies
-    cos and sin (a magnitude correction of rescaled frequencies)."""
+    cos and sin (a magnitude correction of rescaled frequencies).  v_first [T, kv_heads*vdim] (a view with a row
+    stride is fine): the cached value is (1 - v_mix) v + v_mix v_first."""
     assert qkv.dim() == 2 and qkv.stride(1) == 1
     assert qkv.shape[1] >= heads * dim + kv_heads * (dim if v_from_k else dim + vdim)
     assert not v_from_k or vdim == dim
@@ -788,6 +797,9 @@ def rope_append(qkv: torch.Tensor, positions: torch.Tensor, cache_rows: torch.Te
         assert t_ is None or (unit_norm and t_.numel() == dim)
     p.q_norm_w, p.k_norm_w, p.v_from_k = _f32(q_norm_w, "q_norm_w"), _f32(k_norm_w, "k_norm_w"), 1 if v_from_k else 0
     p.rot_layout, p.rot_mscale = 1 if halves else 0, float(mscale)
+    if v_first is not None:
+        assert v_first.shape == (T, kv_heads * vdim) and v_first.stride(1) == 1 and not v_from_k
+        p.v_first, p.ld_vf, p.v_first_dtype, p.v_mix = _p(v_first), v_first.stride(0), _dt(v_first, "v_first"), float(v_mix)
     check(_lib.load().vila_rope_append(C.byref(p), _stream()), "vila_rope_append")
     return q
 
@@ -798,7 +810,8 @@ def paged_attention(q: torch.Tensor, pool: torch.Tensor, page_tables: torch.Tens
                     out: Optional[torch.Tensor] = None, out_dtype=None, max_rows: int = 16,
                     nsplit: int = 1, dist_bias: Optional[torch.Tensor] = None, chunk: int = 0,
                     gate: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0,
-                    talk_after: bool = False, head_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    talk_after: bool = False, head_scale: Optional[torch.Tensor] = None,
+                    softcap: float = 0.0) -> torch.Tensor:
     """Causal grouped-query attention of q fp32 [T, heads*dim] over the paged k | v pool, fp32 scores and
     softmax, optional mixing of the heads' scores (talk fp32 [heads, heads]) and per-head sink logit in
     the denominator.  tiles int32 [n, 4] = (row0, rows <= max_rows, pos0, slot) -> [T, heads*vdim].
@@ -808,7 +821,8 @@ def paged_attention(q: torch.Tensor, pool: torch.Tensor, page_tables: torch.Tens
     row stride is fine): the output of head h is multiplied by sigmoid(gate[t, h]).
     window > 0: a key is seen only when it is less than `window` positions back or among the first `keep_first`
     of its sequence.  talk_after: talk mixes the heads' softmax weights instead of their scores (no sink then).
-    head_scale fp32 [heads]: per-head multiplier of the scores."""
+    head_scale fp32 [heads]: per-head multiplier of the scores.  softcap > 0: every head's own scaled score becomes
+    softcap * tanh(score / softcap) before mixing, bias and softmax."""
     assert q.dtype == torch.float32 and q.is_contiguous() and q.shape[1] == heads * dim
     assert pool.dim() == 2 and pool.is_contiguous() and pool.shape[1] == kv_heads * (dim + vdim)
     if out is None:
@@ -835,6 +849,7 @@ def paged_attention(q: torch.Tensor, pool: torch.Tensor, page_tables: torch.Tens
     if head_scale is not None:
         assert head_scale.numel() == heads
         p.head_scale = _f32(head_scale, "head_scale")
+    p.softcap = float(softcap)
     p.nsplit = max(1, int(nsplit)) if max_rows == 1 else 1
     partial = None
     if p.nsplit > 1:
@@ -971,6 +986,9 @@ def causal_conv_rows(u: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tens
     p.in_dtype, p.w_dtype, p.out_dtype = _dt(u, "u"), _dt(w, "w"), _dt(out, "out")
     p.rows, p.nseq, p.cols, p.taps, p.act = T, seqs.shape[0], Cc, taps, act
     lib = _lib.load()
+    if update_state and p.rows == p.nseq:   # one row per sequence (decoded tokens): output and tail in one launch
+        check(lib.vila_causal_conv_step(C.byref(p), _stream()), "vila_causal_conv_step")
+        return out
     check(lib.vila_causal_conv_rows(C.byref(p), _stream()), "vila_causal_conv_rows")
     if update_state and taps > 1:
         check(lib.vila_causal_conv_state(C.byref(p), _stream()), "vila_causal_conv_state")
@@ -1027,4 +1045,81 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, z: Optio
     p.in_dtype, p.out_dtype = _dt(x, "x"), _dt(out, "out")
     p.nseq, p.C, p.N = seqs.shape[0], Cc, N
     check(_lib.load().vila_selective_scan(C.byref(p), _stream()), "vila_selective_scan")
+    return out
+
+
+# ---- outer-product recurrences (gated delta rule, gated linear attention) and parallel sublayers with channel scales ----
+def delta_scan(qkv: torch.Tensor, a: torch.Tensor, b: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, *, heads: int,
+               kv_heads: int, dim: int, vdim: int, A_log: torch.Tensor, dt_bias: torch.Tensor, q_scale: float,
+               unit_eps: float = 1e-6) -> torch.Tensor:
+    """Gated delta rule per head: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q with unit q (times q_scale) and
+    k, g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b).  qkv [T, kv_heads*dim*2 + heads*vdim] = q | k | v;
+    a, b [T, heads] (views with a row stride are fine); state fp32 [slots, heads, vdim, dim], advanced in place;
+    seqs int32 [n, 4] = (row0, rows, pos0, slot) -> o fp32 [T, heads*vdim]."""
+    T = qkv.shape[0]
+    assert qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] == 2 * kv_heads * dim + heads * vdim
+    assert a.shape == (T, heads) and b.shape == (T, heads) and a.stride(1) == b.stride(1) == 1 and a.dtype == b.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, vdim, dim)
+    assert A_log.numel() == heads and dt_bias.numel() == heads
+    out = torch.empty(T, heads * vdim, dtype=torch.float32, device=qkv.device)
+    p = _lib.DeltaScanParams()
+    p.qkv, p.ld_qkv, p.a, p.ld_a, p.b, p.ld_b = _p(qkv), qkv.stride(0), _p(a), a.stride(0), _p(b), b.stride(0)
+    p.A_log, p.dt_bias = _f32(A_log, "A_log"), _f32(dt_bias, "dt_bias")
+    p.state, p.seqs, p.out, p.ld_out = _p(state), _i32(seqs, "seqs"), _p(out), out.stride(0)
+    p.in_dtype, p.ab_dtype = _dt(qkv, "qkv"), _dt(a, "a")
+    p.nseq, p.H, p.G, p.dim, p.vdim = seqs.shape[0], heads, kv_heads, dim, vdim
+    p.q_scale, p.unit_eps = q_scale, unit_eps
+    check(_lib.load().vila_delta_scan(C.byref(p), _stream()), "vila_delta_scan")
+    return out
+
+
+def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, *,
+             heads: int, dim: int, vdim: int, q_scale: float, tau: float, z_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Gated linear attention per head: S <- diag(alpha) S + k v^T, o = S^T (q_scale q), alpha = sigmoid(z + z_bias)^(1/tau).
+    q, k, z [T, heads*dim], v [T, heads*vdim] (views with a row stride are fine; q, k, v of one dtype); z_bias fp32; state
+    fp32 [slots, heads, vdim, dim], advanced in place; seqs int32 [n, 4] -> o fp32 [T, heads*vdim]."""
+    T = q.shape[0]
+    assert q.shape == k.shape == z.shape == (T, heads * dim) and v.shape == (T, heads * vdim)
+    assert q.stride(1) == k.stride(1) == v.stride(1) == z.stride(1) == 1 and q.dtype == k.dtype == v.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, vdim, dim)
+    assert z_bias is None or z_bias.numel() == heads * dim
+    out = torch.empty(T, heads * vdim, dtype=torch.float32, device=q.device)
+    p = _lib.GlaScanParams()
+    p.q, p.k, p.v, p.z = _p(q), _p(k), _p(v), _p(z)
+    p.ld_q, p.ld_k, p.ld_v, p.ld_z = q.stride(0), k.stride(0), v.stride(0), z.stride(0)
+    p.z_bias = _f32(z_bias, "z_bias")
+    p.state, p.seqs, p.out, p.ld_out = _p(state), _i32(seqs, "seqs"), _p(out), out.stride(0)
+    p.in_dtype, p.z_dtype = _dt(q, "q"), _dt(z, "z")
+    p.nseq, p.H, p.dim, p.vdim, p.q_scale, p.tau = seqs.shape[0], heads, dim, vdim, q_scale, tau
+    check(_lib.load().vila_gla_scan(C.byref(p), _stream()), "vila_gla_scan")
+    return out
+
+
+def gated_head_norm_rows(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, *, heads: int, eps: float, out_dtype=None
+                         ) -> torch.Tensor:
+    """o fp32 [T, heads*vdim] -> rms(o per head) * w [vdim] * silu(gate [T, heads*vdim]) (gate: a view is fine)"""
+    assert o.dtype == torch.float32 and o.is_contiguous() and o.dim() == 2 and o.shape[1] % heads == 0
+    T, vdim = o.shape[0], o.shape[1] // heads
+    assert w.numel() == vdim and gate.shape == o.shape and gate.stride(1) == 1
+    out = torch.empty(o.shape, dtype=out_dtype or gate.dtype, device=o.device)
+    check(_lib.load().vila_gated_head_norm_rows(_p(o), _f32(w, "w"), _p(gate), _dt(gate, "gate"), gate.stride(0), eps, _p(out),
+                                                _dt(out, "out"), T, heads, vdim, _stream()), "vila_gated_head_norm_rows")
+    return out
+
+
+def scaled_residual_norm_rows(x: torch.Tensor, a: torch.Tensor, a_scale: torch.Tensor, b: Optional[torch.Tensor] = None,
+                              b_scale: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None, eps: float = 0.0, *,
+                              out_dtype=None) -> Optional[torch.Tensor]:
+    """x fp32 [rows, cols] (in place) += a_scale * a + b_scale * b (per-channel fp32 scales; b may be None).  With w: also
+    -> rmsnorm(x) * w in out_dtype, the operand of the sublayers that read x next; without: -> None."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2
+    rows, cols = x.shape
+    assert a.shape == (rows, cols) and a.stride(1) == 1 and a_scale.numel() == cols
+    if b is not None:
+        assert b.shape == (rows, cols) and b.stride(1) == 1 and b_scale is not None and b_scale.numel() == cols
+    out = torch.empty(rows, cols, dtype=out_dtype or x.dtype, device=x.device) if w is not None else None
+    check(_lib.load().vila_scaled_residual_norm_rows(
+        _p(x), _p(a), _dt(a, "a"), a.stride(0), _f32(a_scale, "a_scale"), _p(b), _dt(b, "b") if b is not None else 0,
+        b.stride(0) if b is not None else 0, _f32(b_scale, "b_scale"), _f32(w, "w"), eps, _p(out),
+        _dt(out, "out") if out is not None else 0, rows, cols, _stream()), "vila_scaled_residual_norm_rows")
     return out
