@@ -1846,6 +1846,243 @@ def run_window_lm(args):
     print(json.dumps(res))
 
 
+# ------------------------------------------------------------------------------------------------
+# --workload delta_lm: the Bivizen language model (gated delta rule, gated linear attention, capped rotary attention,
+# parallel clamped-GLU feed-forwards) next to Nusovik (the closest model of the package: same engine, recurrent mixers
+# with an fp32 state per slot behind a short convolution, grouped-query attention with an output gate, dense
+# feed-forwards) at equal width / heads / vocabulary, random weights, bf16.  The scans are set beside ssd_scan and
+# Moronex's hgrn2_scan on states of the same size.
+# ------------------------------------------------------------------------------------------------
+def delta_lm_config(z):
+    W, H, G = z["width"], z["heads"], z["kv_heads"]
+    ff = {"ff": z["ff"] * 2 // 3 // 64 * 64, "kind": "dense", "limit": 7.0}      # gated: three matrices of 2/3 the width
+    att = {"dim": 128, "heads": H, "kv_heads": G, "rot": {"base": 250000.0, "dims": 128}, "scale": 128 ** -0.5,
+           "softcap": 30.0, "v_mix": True, "vdim": 128}
+    gla = {"dim": 128, "heads": H, "tau": 8.0, "vdim": 128}
+    delta = {"conv": 4, "dim": 128, "heads": H, "kv_heads": H // 2, "vdim": 128}
+    return {"architecture": "Bivizen", "layers": [{"type": t, "mixer": dict(m), "mlp": dict(ff)} for t, m in (
+        ("attention", att), ("gla", gla), ("delta", delta), ("attention", att))],
+        "norm": {"eps": 1e-5}, "vocab": z["vocab"], "width": W}
+
+
+def delta_lm_block(args, peaks):
+    import torch
+
+    from vila_b200 import ops
+    from vila_b200.model import BivizenConfig, BivizenForCausalLM, NusovikConfig, NusovikForCausalLM
+    from vila_b200.serving import TokenEngine
+    dev = torch.device("cuda:0")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+
+    def timed(fn, reps=args.steps, warm=max(3, args.warmup), setup=None):
+        ts = []
+        for i in range(warm + reps):
+            if setup is not None:
+                setup()
+            flush.fill_(i & 255)     # evict L2 (126 MB) between iterations
+            a, b = ev(), ev()
+            torch.cuda.synchronize()
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            if i >= warm:
+                ts.append(a.elapsed_time(b))
+        ts.sort()
+        return ts[len(ts) // 2]
+
+    def timed_op(fn):
+        """captured once, timed as a graph replay: the device time of the op's launches, not the host time around them"""
+        fn()
+        fn()
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            fn()
+        return timed(g.replay)
+
+    S, B, CTX, NEW = 2048, 8, 1024, 32
+    tf, gbs = peaks["bf16_tflops"], peaks["hbm_gbs"]
+    bf = torch.bfloat16
+    out = {}
+    t00 = time.time()
+
+    def log(msg):
+        print("[delta_lm %6.1fs] %s" % (time.time() - t00, msg), file=sys.stderr, flush=True)
+
+    def engine_numbers(lm, prompt):
+        eng = TokenEngine(lm, max_tokens=B * (CTX + 4 * NEW + 64), slots=B)
+        t_pre = timed(lambda: eng.step([("p", prompt, [S - 1])]), setup=lambda: eng.release("p"))
+        eng.release("p")
+        for b in range(B):
+            eng.step([(b, prompt[:CTX], [])])
+        step_in = [[(b, [int(prompt[(k * 7 + b) % S])], [0]) for b in range(B)] for k in range(NEW)]
+
+        def decode_run():
+            for k in range(NEW):
+                eng.step(step_in[k])
+        t_dec = timed(decode_run, reps=3, warm=1)     # contexts grow CTX .. CTX + 4 * NEW: fits the reserve
+        for b in range(B):
+            eng.release(b)
+        n = sum(v.numel() for v in lm.weights.values())
+        return eng, {"params_m": n / 1e6, "prefill_tok_s": S / t_pre * 1e3, "prefill_ms": t_pre,
+                     "decode_tok_s": B * NEW / t_dec * 1e3, "decode_ms_per_step": t_dec / NEW}
+
+    def flops(t, fl):
+        return {"ms": t, "tflops": fl / t / 1e9, "of_bf16_peak": fl / t / 1e9 / tf}
+
+    def bytes_(t, by):
+        return {"ms": t, "gbs": by / t / 1e6, "of_hbm": by / t / 1e6 / gbs}
+
+    for name, z in SSM_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        W, H, G = z["width"], z["heads"], z["kv_heads"]
+        g = torch.Generator().manual_seed(0)
+        prompt = torch.randint(0, z["vocab"], (S,), generator=g).tolist()
+        log("size %s: bivizen" % name)
+        lm = BivizenForCausalLM(BivizenConfig.from_dict(delta_lm_config(z)), dev, bf).init_random(0, on_device=True)
+        eng, res_new = engine_numbers(lm, prompt)
+        log("size %s: nusovik" % name)
+        tw = NusovikForCausalLM(NusovikConfig.from_dict(ssm_lm_config(z)), dev, bf).init_random(0, on_device=True)
+        eng2, res_old = engine_numbers(tw, prompt)
+        # ---- kernel beside the like kernel ---------------------------------------------------------------
+        log("kernel ledger")
+        led = {}
+        La, Lg, Ld, Nl = lm.layers[0], lm.layers[1], lm.layers[2], tw.layers[1]
+        sq1 = torch.tensor([[0, S, 0, 0]], dtype=torch.int32, device=dev)
+        sqB = torch.tensor([(b, 1, CTX, b) for b in range(B)], dtype=torch.int32, device=dev)
+        sqP = torch.tensor([(b * (S // B), S // B, 0, b) for b in range(B)], dtype=torch.int32, device=dev)
+        rs1, rsB = torch.zeros(S, dtype=torch.int32, device=dev), torch.arange(B, dtype=torch.int32, device=dev)
+        # scans over states [H, 128, 128]: flops counted as 2 per multiply-add of the recurrence's own products
+        D = 128
+        KH = H // 2
+        std, stg = eng.cache.state[(2, "scan")], eng.cache.state[(1, "scan")]
+        stx = torch.zeros(B, H, D, D, device=dev)
+        wide = (torch.randn(S, 6 * H * D + 8, device=dev) * 0.5).to(bf)
+        ab = torch.randn(S, 2 * H, device=dev).to(bf)
+        par = torch.zeros(H, device=dev)
+        zero = torch.zeros(H * D, device=dev)
+        for rows, sq, tag in ((S, sq1, "prefill, one %d-row prompt" % S), (S, sqP, "prefill, %d prompts of %d rows" % (B, S // B)),
+                              (B, sqB, "decode, %d rows" % B)):
+            nseq = sq.shape[0]
+            x = wide[:rows]
+            rate = (lambda t, fl, by: bytes_(t, by)) if rows == B else (lambda t, fl, by: {"ms": t, "tflops_fp32": fl / t / 1e9})
+            st_by = 2 * nseq * H * D * D * 4
+            t = timed_op(lambda: ops.delta_scan(x[:, :2 * KH * D + H * D], ab[:rows, :H], ab[:rows, H:], std, sq, heads=H,
+                                                kv_heads=KH, dim=D, vdim=D, A_log=Ld.A_log, dt_bias=Ld.dt_bias, q_scale=D ** -0.5))
+            led["delta_scan " + tag] = rate(t, 8.0 * rows * H * D * D, st_by + rows * H * D * (4 + 4))
+            t = timed_op(lambda: ops.gla_scan(x[:, :H * D], x[:, H * D:2 * H * D], x[:, 2 * H * D:3 * H * D],
+                                              x[:, 3 * H * D:4 * H * D], stg, sq, heads=H, dim=D, vdim=D, q_scale=D ** -0.5,
+                                              tau=8.0, z_bias=Lg.a2_b))
+            led["gla_scan " + tag] = rate(t, 6.0 * rows * H * D * D, st_by + rows * H * D * (8 + 4))
+            t = timed_op(lambda: ops.ssd_scan(x[:, :H * D + 2 * KH * D], ab[:rows, :H], None, stx, sq, heads=H, vdim=D, nstate=D,
+                                              groups=KH, dt_bias=par, A_log=par, D=par))
+            led["nusovik ssd_scan, the same state " + tag] = rate(t, 6.0 * rows * H * D * D, st_by + rows * H * D * (4 + 4))
+            t = timed_op(lambda: ops.hgrn2_scan(x, stx, sq, heads=H, dim=D, vdim=D, q_off=0, f_off=H * D, v_off=2 * H * D,
+                                                f_bias=zero, lower=zero))
+            led["moronex hgrn2_scan, the same state " + tag] = rate(t, 6.0 * rows * H * D * D, st_by + rows * H * D * (6 + 4))
+        # attention: the paged kernels with this model's options, with none, and with Nusovik's
+        page, npg = eng.cache.page, eng.cache.n_pages
+        pool = eng.cache.latent[0]
+        pt = torch.arange(npg, dtype=torch.int32, device=dev).view(1, -1).repeat(B, 1).contiguous()
+        tiles = torch.tensor([(o, 16, o, 0) for o in range(0, S, 16)], dtype=torch.int32, device=dev)
+        q = torch.randn(S, H * D, device=dev)
+        gate = torch.randn(S, H, device=dev).to(bf)
+        akw = dict(heads=H, kv_heads=G, dim=D, vdim=D, page=page, scale=0.088)
+        fl = H * (S * (S + 1) / 2) * 4.0 * D
+        att = lambda t, f: {"ms": t, "tflops_fp32": f / t / 1e9}
+        t = timed_op(lambda: ops.paged_attention(q, pool, pt, tiles, max_rows=16, softcap=30.0, gate=gate, **akw))
+        led["paged_attention prefill: capped scores + gate"] = att(t, fl)
+        t = timed_op(lambda: ops.paged_attention(q, pool, pt, tiles, max_rows=16, **akw))
+        led["paged_attention prefill: plain causal"] = att(t, fl)
+        ck = z["chunk"]
+        t = timed_op(lambda: ops.paged_attention(q, pool, pt, tiles, max_rows=16, sink=Nl.sink, dist_bias=Nl.dist_bias, chunk=ck,
+                                                 gate=gate, **akw))
+        led["nusovik paged_attention prefill: chunk %d + distance bias + sink + gate" % ck] = att(t, H * sum((p % ck) + 1 for p in range(S)) * 4.0 * D)
+        dt_ = torch.tensor([(b, 1, CTX - 1, b) for b in range(B)], dtype=torch.int32, device=dev)
+        pt2 = ((torch.arange(B, device=dev, dtype=torch.int32)[:, None] * (CTX // page) +
+                torch.arange(npg, device=dev, dtype=torch.int32)[None]) % npg).contiguous()
+        ns = eng.cache.decode_splits
+        t = timed_op(lambda: ops.paged_attention(q[:B], pool, pt2, dt_, max_rows=1, nsplit=ns, softcap=30.0, gate=gate[:B], **akw))
+        led["paged_attention decode: capped scores + gate (8 x 1024 keys)"] = bytes_(t, B * CTX * G * 2 * D * 2)
+        t = timed_op(lambda: ops.paged_attention(q[:B], pool, pt2, dt_, max_rows=1, nsplit=ns, **akw))
+        led["paged_attention decode: plain causal (8 x 1024 keys)"] = bytes_(t, B * CTX * G * 2 * D * 2)
+        ar = torch.arange(S, dtype=torch.int32, device=dev)
+        qkv = wide[:, :(H + 2 * G) * D]
+        vf = wide[:, 4 * H * D:4 * H * D + G * D]
+        by = S * ((H + 2 * G) * D * 2 + H * D * 4 + 2 * G * D * 2)
+        t = timed_op(lambda: ops.rope_append(qkv, ar, ar, pool, heads=H, kv_heads=G, dim=D, vdim=D, inv_freq=La.inv_freq,
+                                             unit_norm=False, eps=0.0, halves=True, v_first=vf, v_mix=0.4))
+        led["rope_append: rotary in halves + value mixing + k | v append (2048 rows)"] = bytes_(t, by + S * G * D * 2)
+        t = timed_op(lambda: ops.rope_append(wide[:, :(H + G) * D], ar, ar, pool, heads=H, kv_heads=G, dim=D, vdim=D, inv_freq=None,
+                                             unit_norm=True, eps=1e-5, q_norm_w=Nl.q_norm, k_norm_w=Nl.k_norm, v_from_k=True))
+        led["nusovik head norm + k | v append (2048 rows)"] = bytes_(t, S * ((H + G) * D * 2 + H * D * 4 + 2 * G * D * 2))
+        # convolution
+        ch = 2 * KH * D + H * D
+        cst = eng.cache.state[(2, "conv")]
+        t = timed_op(lambda: ops.causal_conv_rows(wide[:, :ch], Ld.conv, None, cst, sq1, rs1, act=ops.CONV_SILU, out_dtype=bf))
+        led["causal_conv_rows + tail update, 2 x width channels, 4 taps, SiLU (2048 rows)"] = bytes_(t, S * ch * 4)
+        t = timed_op(lambda: ops.causal_conv_rows(wide[:B, :ch], Ld.conv, None, cst, sqB, rsB, act=ops.CONV_SILU, out_dtype=bf))
+        led["causal_conv_step, 2 x width channels, 4 taps, SiLU (decode, 8 rows)"] = bytes_(t, B * ch * (4 + 24) + ch * 16)
+        t = timed_op(lambda: ops.causal_conv_rows(wide[:B, :ch], Ld.conv, None, cst, sqB, rsB, act=ops.CONV_SILU, out_dtype=bf,
+                                                  update_state=False))
+        led["the same convolution without the tail update (decode, 8 rows; the tail was a second launch)"] = bytes_(t, B * ch * (4 + 12) + ch * 16)
+        # row kernels
+        o = torch.randn(S, H * D, device=dev)
+        gt = wide[:, :H * D]
+        t = timed_op(lambda: ops.gated_head_norm_rows(o, Lg.norm, gt, heads=H, eps=1e-5, out_dtype=bf))
+        led["gated_head_norm_rows: per-head norm, weight, SiLU gate (2048 rows)"] = bytes_(t, S * H * D * (4 + 2 + 2))
+        t = timed_op(lambda: ops.rmsnorm_rows(o.view(-1, D), Lg.norm, 1e-5, out_dtype=bf))
+        led["rmsnorm_rows per head, no gate (2048 rows)"] = bytes_(t, S * H * D * (4 + 2))
+        x = torch.randn(S, W, device=dev)
+        y1, y2 = torch.randn(S, W, device=dev).to(bf), torch.randn(S, W, device=dev).to(bf)
+        t = timed_op(lambda: ops.scaled_residual_norm_rows(x, y1, La.ls1, y2, La.ls2, La.norm1, 1e-5, out_dtype=bf))
+        led["scaled_residual_norm_rows: two branches with channel scales + next norm (2048 rows)"] = bytes_(t, S * W * (8 + 2 + 2 + 2))
+        t = timed_op(lambda: ops.branch_norm_residual(x, y1, Nl.norm1, 1e-5, a_scale=1.0, b=y2, b_scale=1.0, copy_dtype=bf))
+        led["nusovik branch_norm_residual: two branches + bf16 copy (2048 rows)"] = bytes_(t, S * W * (8 + 2 + 2 + 2))
+        # projections
+        hb = torch.randn(S, W, device=dev).to(bf)
+        fl = 2.0 * S * W * La.gu.shape[0]
+        t = timed_op(lambda: ops.linear_any(hb, La.gu, glu_clamp=(1.702, 7.0)))
+        led["gate | up projection, clamped-GLU epilogue (tcgen05)"] = flops(t, fl)
+        t = timed_op(lambda: ops.linear_any(hb, La.gu, swiglu=True))
+        led["the same projection, SwiGLU epilogue (tcgen05)"] = flops(t, fl)
+        t = timed_op(lambda: ops.linear_any(hb[:B], La.gu, glu_clamp=(1.702, 7.0)))
+        led["gate | up projection decode, clamped-GLU epilogue (8 rows)"] = bytes_(t, La.gu.numel() * 2)
+        t = timed_op(lambda: ops.linear_any(hb[:B], La.gu, swiglu=True))
+        led["the same projection decode, SwiGLU epilogue (8 rows)"] = bytes_(t, La.gu.numel() * 2)
+        rk = hb[:, :Lg.a2.shape[1]].contiguous()
+        t = timed_op(lambda: ops.linear_any(rk, Lg.a2))
+        led["decay projection from rank %d (2048 rows)" % Lg.a2.shape[1]] = bytes_(t, S * H * D * 2)
+        out[name] = {"bivizen": res_new, "nusovik": res_old, "kernels": led}
+        del lm, tw, eng, eng2
+        torch.cuda.empty_cache()
+    return {"workload": "delta_lm: 4 Bivizen layers (capped rotary GQA with value mixing; gated linear attention; gated delta "
+                        "rule; attention; each with a parallel clamped-GLU feed-forward) vs 4 Nusovik layers (selective scan; "
+                        "chunked sink attention + scalar-decay scan in parallel + squared-ReLU feed-forward; twice) of equal "
+                        "width / heads / vocabulary; prefill: one %d-token prompt; decode: %d sequences x %d-token context, %d "
+                        "steps" % (S, B, CTX, NEW),
+            "dtype": "bf16", "data": "synthetic (random weights, random ids)",
+            "l2_policy": "256 MB buffer written between timed iterations",
+            "kernel_ledger_timing": "each op captured in a CUDA graph, one replay per timed iteration", "peaks": peaks, "sizes": out}
+
+
+def run_delta_lm(args):
+    import torch
+    assert torch.cuda.is_available(), "bench.py --workload delta_lm needs a GPU"
+    import faulthandler
+    faulthandler.dump_traceback_later(int(os.environ.get("VILA_BENCH_WATCHDOG_S", "480")), exit=True)
+    peaks = read_peaks()
+    with ClockSampler(0) as cs:
+        res = delta_lm_block(args, peaks)
+    res["clocks"] = cs.summary()
+    from vila_b200 import _lib
+    res["gpu_launches"] = _lib.LAUNCHES
+    print(json.dumps(res))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1860,12 +2097,12 @@ def main():
     ap.add_argument("--sp-steps", type=int, default=10)
     ap.add_argument("--profile", action="store_true",
                     help="profiling aid (ncu): 1 warm-up, 8 new tokens, no extra blocks; NOT a valid bench number")
-    ap.add_argument("--sizes", default="", help="hybrid_lm / parallel_lm / ssm_lm / window_lm: comma-separated subset of the workload's sizes ("
+    ap.add_argument("--sizes", default="", help="hybrid_lm / parallel_lm / ssm_lm / window_lm / delta_lm: comma-separated subset of the workload's sizes ("
                     + ",".join(HYBRID_SIZES) + " / " + ",".join(PARALLEL_SIZES) + ")")
-    ap.add_argument("--workload", default="headline", choices=["headline", "hybrid_lm", "parallel_lm", "ssm_lm", "window_lm"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "hybrid_lm", "parallel_lm", "ssm_lm", "window_lm", "delta_lm"],
                     help="headline (default): the NVILA-8B serving step; hybrid_lm: Moronex vs Qwen2 at equal size; "
                          "parallel_lm: Lufatar vs Moronex at equal size; ssm_lm: Nusovik vs Moronex at equal size; "
-                         "window_lm: Ludazen vs Lufatar at equal size")
+                         "window_lm: Ludazen vs Lufatar at equal size; delta_lm: Bivizen vs Nusovik at equal size")
     args = ap.parse_args()
     if args.workload == "hybrid_lm":
         return run_hybrid_lm(args)
@@ -1875,6 +2112,8 @@ def main():
         return run_ssm_lm(args)
     if args.workload == "window_lm":
         return run_window_lm(args)
+    if args.workload == "delta_lm":
+        return run_delta_lm(args)
     if args.profile:
         global NEW_TOKENS
         NEW_TOKENS = 8

@@ -13,11 +13,11 @@
 //   delta:  S_new^T q = g (S^T q) + (k . q) u        so S^T k and S^T q are reduced together
 //   gla:    S_new^T q = S^T (alpha q) + (k . q) v    so the state update does not wait for the reduction
 //
-// Grid (sequence, head, COLS columns of vdim), 8 warps.  Warps 0-3 own the state: R lanes share CPT columns, lane r
+// Grid (sequence, head, COLS columns of vdim).  Warps 0-3 own the state: R lanes share CPT columns, lane r
 // keeps the float4 pieces r, r + R, .. of a column in registers (state layout [.., vdim, dim]: coalesced loads, and
 // the lanes' reads of a token's k / q from shared memory fall into consecutive banks).  The 2 CPT (or CPT) column
 // sums are reduced over the R lanes with a transposing tree: every step halves the number of values a lane carries.
-// Warps 4-7 stage the next 16 tokens (load, unit norms or decays, k . q, fp32 into the other shared-memory buffer)
+// The other 4 or 8 warps stage the next 16 tokens (load, unit norms or decays, k . q, fp32 into the other shared-memory buffer)
 // and write the previous 16 tokens' outputs while the owners run; one barrier per 16 tokens.
 // A column's sum runs in the same order whatever CPT is, and time runs in order: a row's result depends neither on
 // the batch nor on how its sequence was cut into steps.
@@ -29,8 +29,7 @@
 namespace vb {
 namespace {
 
-constexpr int kThreads = 256;
-constexpr int kOwnerWarps = 4, kStageWarps = 4;
+constexpr int kOwnerWarps = 4;
 constexpr int kChunk = 16;   // tokens per stage
 
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
@@ -105,8 +104,8 @@ struct ScanArgs {
   int vec_qk, vec_a;            // four-element loads of q | k and of z are aligned
 };
 
-template <bool DELTA, int R, int KPT, int CPT>
-__global__ void __launch_bounds__(kThreads) outer_scan_kernel(const ScanArgs p) {
+template <bool DELTA, int R, int KPT, int CPT, int kStageWarps>
+__global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_kernel(const ScanArgs p) {
   extern __shared__ __align__(16) float sm[];
   constexpr int NP = R * KPT;                       // key channels the owners cover
   constexpr int NQ = KPT / 4;                       // float4 pieces per lane
@@ -116,7 +115,8 @@ __global__ void __launch_bounds__(kThreads) outer_scan_kernel(const ScanArgs p) 
   constexpr int NVEC = DELTA ? 2 : 3;               // staged vectors per token: k, q (, alpha)
   constexpr int TOK = NVEC * NP;
   constexpr int NG = NP > 128 ? NP / 128 : 1;       // four-element pieces a staging lane handles per vector
-  constexpr int TB = NG == 1 ? 4 : (NG == 2 ? 2 : 1);   // tokens a staging warp has in flight
+  constexpr int TPW = kChunk / kStageWarps;         // tokens of a stage per staging warp
+  constexpr int TB = NG == 1 ? TPW : (NG == 2 ? 2 : 1);   // of which it has so many in flight
   float* vec_s = sm;                                // [2][kChunk][NVEC][NP]
   float* v_s = vec_s + 2 * kChunk * TOK;            // [2][kChunk][COLS]
   float* y_s = v_s + 2 * kChunk * COLS;             // [2][kChunk][COLS]
@@ -164,7 +164,7 @@ __global__ void __launch_bounds__(kThreads) outer_scan_kernel(const ScanArgs p) 
         rb = ld_raw(p.b, adt, static_cast<size_t>(row0 + t0 + st) * p.ldb + h);
       }
 #pragma unroll 1
-      for (int tb = 0; tb < kChunk / kStageWarps; tb += TB) {
+      for (int tb = 0; tb < TPW; tb += TB) {
         uint4 rk[TB][NG], rq[TB][NG], rz[TB][NG];
 #pragma unroll
         for (int u = 0; u < TB; ++u) {
@@ -393,13 +393,16 @@ int launch_scan(const ScanArgs& p, int nseq, cudaStream_t stream) {
   constexpr int NP = R * KPT, COLS = kOwnerWarps * (32 / R) * CPT;
   constexpr size_t smem = sizeof(float) * (2 * kChunk * (DELTA ? 2 : 3) * NP + 4 * kChunk * COLS + 2 * kChunk * 4);
   static_assert(smem <= 224 * 1024, "outer_scan: shared memory");
-  auto kern = outer_scan_kernel<DELTA, R, KPT, CPT>;
+  // the staging work of a token is the same for 2 as for 4 columns per group: twice the warps for the narrow form,
+  // where an SM holds one or two CTAs, fewer for the wide one, where CTAs share it
+  constexpr int SW = CPT == 4 ? 4 : 8;
+  auto kern = outer_scan_kernel<DELTA, R, KPT, CPT, SW>;
   static PerDeviceOnce attr_once;
   if (smem > 48 * 1024 && attr_once.first())
     VB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   const dim3 grid(nseq, p.H, (p.vdim + COLS - 1) / COLS);
   VB_CHECK(grid.y <= 65535 && grid.z <= 65535, "outer_scan: H=%d vdim=%d", p.H, p.vdim);
-  VB_CUDA(launch_serial(kern, grid, dim3(kThreads), smem, stream, p));
+  VB_CUDA(launch_serial(kern, grid, dim3(32 * (kOwnerWarps + SW)), smem, stream, p));
   return 0;
 }
 
