@@ -2001,6 +2001,13 @@ def delta_lm_block(args, peaks):
         t = timed_op(lambda: ops.paged_attention(q, pool, pt, tiles, max_rows=16, sink=Nl.sink, dist_bias=Nl.dist_bias, chunk=ck,
                                                  gate=gate, **akw))
         led["nusovik paged_attention prefill: chunk %d + distance bias + sink + gate" % ck] = att(t, H * sum((p % ck) + 1 for p in range(S)) * 4.0 * D)
+        # every query head with its own key head, beside Moronex's kernel for that layout
+        mpool = torch.randn(S, H * 2 * D, device=dev).to(bf)
+        t = timed_op(lambda: ops.paged_attention(q, mpool, pt, tiles, max_rows=16, softcap=30.0, gate=gate, **dict(akw, kv_heads=H)))
+        led["paged_attention prefill: capped scores + gate, a key head per query head"] = att(t, fl)
+        qb = q.to(bf)
+        t = timed_op(lambda: ops.sink_attention(qb, mpool[:, :H * D], mpool[:, H * D:], tiles, heads=H, scale=0.088, gate=gate))
+        led["moronex sink_attention prefill, a key head per query head"] = att(t, fl)
         dt_ = torch.tensor([(b, 1, CTX - 1, b) for b in range(B)], dtype=torch.int32, device=dev)
         pt2 = ((torch.arange(B, device=dev, dtype=torch.int32)[:, None] * (CTX // page) +
                 torch.arange(npg, device=dev, dtype=torch.int32)[None]) % npg).contiguous()
