@@ -1856,7 +1856,7 @@ def run_window_lm(args):
 def delta_lm_config(z):
     W, H, G = z["width"], z["heads"], z["kv_heads"]
     ff = {"ff": z["ff"] * 2 // 3 // 64 * 64, "kind": "dense", "limit": 7.0}      # gated: three matrices of 2/3 the width
-    att = {"dim": 128, "heads": H, "kv_heads": G, "rot": {"base": 250000.0, "dims": 128}, "scale": 128 ** -0.5,
+    att = {"dim": 128, "heads": H, "kv_heads": G, "rot": {"base": 500000.0, "dims": 128}, "scale": 128 ** -0.5,
            "softcap": 30.0, "v_mix": True, "vdim": 128}
     gla = {"dim": 128, "heads": H, "tau": 8.0, "vdim": 128}
     delta = {"conv": 4, "dim": 128, "heads": H, "kv_heads": H // 2, "vdim": 128}
