@@ -66,9 +66,8 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
-// ---- activations (shared by the GEMM / GEMV epilogues).  The division is the fast one
-// (MUFU.RCP + FMUL, ~1 ulp): the IEEE fp32 division's slow path cost ~20 instructions per element
-// in the epilogues, and every result is rounded to bf16 right after.
+// ---- activations (shared by the GEMM / GEMV epilogues).  They divide with __fdividef, which costs less than
+// the correctly rounded division; every result is rounded to bf16 right after.
 __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   // gelu_pytorch_tanh: 0.5 x (1 + tanh( sqrt(2/pi) (x + 0.044715 x^3) ))
