@@ -481,6 +481,13 @@ int vila_sink_attention(const vila_sink_attn_params* p, void* stream);
  *   multiplied by in_scale[a_rows ? a_rows[i] : i] BEFORE bias and activation, which is the layer applied
  *   to the scaled input row (a routing weight on an expert's input rather than on its output). */
 #define VILA_ACT_XIELU 5
+/* act = VILA_ACT_SOFTCAP (vila_glinear only): cap * tanh(z / cap), cap = act_pos of vila_glinear_ext */
+#define VILA_ACT_SOFTCAP 6
+/* act = VILA_ACT_SIGMOID: only where a gate's activation is chosen (vila_gated_head_norm_act_rows) */
+#define VILA_ACT_SIGMOID 7
+/* epilogue (flags) of vila_linear_act and vila_glinear: weight rows interleaved (gate_0, up_0, ...) as for
+ * VILA_FLAG_SWIGLU, out = gelu_tanh(z_gate) * z_up with N / 2 columns (vila_linear_act: N a multiple of 32) */
+#define VILA_FLAG_GEGLU 8
 typedef struct vila_glinear_ext {
   float act_alpha, act_limit;
   float act_pos, act_neg;
@@ -546,6 +553,9 @@ typedef struct vila_rope_append_params {
   int64_t ld_vf;
   int32_t v_first_dtype;
   float v_mix;
+  /* maps == 2: every q and k head comes as two maps of `dim` columns side by side (differential attention), values stay
+   * one head each: q_out [T, H * 2 * dim], pool row k (G * 2 * dim) | v (G * vdim); 0 counts as 1; not with v_from_k */
+  int32_t maps;
 } vila_rope_append_params;
 int vila_rope_append(const vila_rope_append_params* p, void* stream);
 
@@ -588,6 +598,12 @@ typedef struct vila_paged_attn_params {
   /* softcap > 0: every head's own score becomes softcap * tanh(score / softcap), after scale and head_scale and
    * before mixing, bias and softmax; 0: off */
   float softcap;
+  /* maps == 2: differential attention.  q is [T, H * 2 * dim], pool rows are k (G * 2 * dim) | v (G * vdim); map m of head
+   * h attends with key head (h / (H / G), m) to value head h / (H / G), giving a_m, and
+   *   o = a_0 - diff_lambda a_1;  out_h = o / sqrt(mean(o^2) + diff_eps) * diff_scale  (mean over vdim), then the gate.
+   * partial is fp32 [T, nsplit, 2 H, vdim + 2].  No talk, sink, dist_bias or head_scale.  0 counts as 1. */
+  int32_t maps;
+  float diff_lambda, diff_scale, diff_eps;
 } vila_paged_attn_params;
 int vila_paged_attention(const vila_paged_attn_params* p, void* stream);
 
@@ -773,6 +789,75 @@ typedef struct vila_gla_scan_params {
   float q_scale, tau;
 } vila_gla_scan_params;
 int vila_gla_scan(const vila_gla_scan_params* p, void* stream);
+
+/* vila_decay_scan — linear attention with one constant decay per head (lightning attention), per head:
+ *   S <- decay_h S + k v^T;  out = S^T (q_scale q);  silu != 0: SiLU is taken on q, k and v first (fp32)
+ * q and k rows hold H heads of dim, v rows H heads of vdim.  out fp32 [rows, ld_out]. */
+typedef struct vila_decay_scan_params {
+  const void *q, *k, *v;
+  int64_t ld_q, ld_k, ld_v;
+  const float* decay; /* [H] */
+  float* state;
+  const int32_t* seqs;
+  float* out;
+  int64_t ld_out;
+  int32_t in_dtype, nseq, H, dim, vdim, silu;
+  float q_scale;
+} vila_decay_scan_params;
+int vila_decay_scan(const vila_decay_scan_params* p, void* stream);
+
+/* Router of routed experts with group-limited choice.  z = w x (fp32), s = sigmoid(z) or softmax(z) over all `experts`
+ * outputs, choice = s + correction (NULL: none); the outputs form `groups` equal groups of neighbours, a group's score is
+ * its largest choice value (group_top == 1) or the sum of its two largest (group_top == 2; its only one if it has one),
+ * only the `keep` best groups can be chosen; the `top` largest choice values win (ties: the lower index);
+ * weight = scale * s of the chosen, not renormalised.  gate_w != NULL: gate[r] = sigmoid(gate_w . x[r]) as well (a shared
+ * expert's gate, read from the same rows).  idx / weight are [rows, top]. */
+#define VILA_SCORE_SIGMOID 0
+#define VILA_SCORE_SOFTMAX 1
+typedef struct vila_moe_route_params {
+  const void* x;
+  int64_t ldx;
+  const float* w;          /* [experts, cols] */
+  const float* correction; /* [experts] or NULL */
+  const float* gate_w;     /* [cols] or NULL */
+  int32_t* idx;
+  float* weight;
+  float* gate; /* [rows] */
+  int32_t x_dtype, rows, cols, experts, top, groups, keep, score, group_top;
+  float scale;
+} vila_moe_route_params;
+int vila_moe_route_scores(const vila_moe_route_params* p, void* stream);
+
+/* Parallel-sublayer residual and the next Dynamic Tanh norms in one elementwise pass over fp32 rows x:
+ *   x[r] = table[ids[r]] (table != NULL) or x[r] as it is
+ *   f    = b[r] * (b_gate ? b_gate[r] : 1) + sum_{j < n_partials} (idx[r, j] < experts ? part[r * n_partials + j]
+ *                                                                                      : weight[r, j] * h[r])
+ *   x[r] += mult * (a_scale * a[r] + b_scale * f)        (a, b, part may be NULL; idx NULL: every partial is read)
+ *   out_k[r] = tanh(alpha_k x[r]) * w_k + bias_k         for k < n_out (0, 1 or 2), contiguous [rows, cols] in out_dtype
+ * (identity experts: an index from `experts` on stands for the row h itself).  x is written when anything was added to it or
+ * it came from the table. */
+typedef struct vila_tanh_residual_params {
+  float* x;
+  const void* table;
+  const int32_t* ids;
+  const void *a, *b, *part, *h;
+  int64_t lda, ldb, ldp, ldh;
+  const float *a_scale, *b_scale, *b_gate;
+  const int32_t* idx;
+  const float* weight;
+  const float* w[2];
+  const float* bias[2];
+  void* out[2];
+  float alpha[2];
+  float mult;
+  int32_t table_dtype, a_dtype, b_dtype, part_dtype, h_dtype, out_dtype, rows, cols, n_partials, experts, n_out;
+} vila_tanh_residual_params;
+int vila_tanh_residual_rows(const vila_tanh_residual_params* p, void* stream);
+
+/* vila_gated_head_norm_rows with the gate's activation chosen: VILA_ACT_SILU or VILA_ACT_SIGMOID.  H = 1, vdim = all columns:
+ * one norm over a whole row. */
+int vila_gated_head_norm_act_rows(const float* o, const float* w, const void* gate, int gate_dtype, int64_t ldg, float eps,
+                                  void* out, int out_dtype, int rows, int H, int vdim, int gate_act, void* stream);
 
 /* Read-out of a recurrent mixer: out[t, h, :] = rms(o[t, h, :]) * w * silu(gate[t, h, :]), rms(v) = v / sqrt(mean(v^2)
  * + eps) over the head's vdim columns, w [vdim] shared by the heads.  o and out are [rows, H * vdim] contiguous. */

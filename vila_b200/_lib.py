@@ -137,6 +137,7 @@ class RopeAppendParams(C.Structure):
         ("q_norm_w", c_void_p), ("k_norm_w", c_void_p), ("v_from_k", C.c_int32),
         ("rot_layout", C.c_int32), ("rot_mscale", c_float),
         ("v_first", c_void_p), ("ld_vf", c_i64), ("v_first_dtype", C.c_int32), ("v_mix", c_float),
+        ("maps", C.c_int32),
     ]
 
 
@@ -151,6 +152,7 @@ class PagedAttnParams(C.Structure):
         ("dist_rows", C.c_int32), ("chunk", C.c_int32), ("gate_dtype", C.c_int32),
         ("window", C.c_int32), ("keep_first", C.c_int32), ("talk_after", C.c_int32), ("head_scale", c_void_p),
         ("softcap", c_float),
+        ("maps", C.c_int32), ("diff_lambda", c_float), ("diff_scale", c_float), ("diff_eps", c_float),
     ]
 
 
@@ -199,6 +201,37 @@ class GlaScanParams(C.Structure):
         ("out", c_void_p), ("ld_out", c_i64),
         ("in_dtype", C.c_int32), ("z_dtype", C.c_int32), ("nseq", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32),
         ("vdim", C.c_int32), ("q_scale", c_float), ("tau", c_float),
+    ]
+
+
+class DecayScanParams(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("ld_q", c_i64), ("ld_k", c_i64), ("ld_v", c_i64),
+        ("decay", c_void_p), ("state", c_void_p), ("seqs", c_void_p), ("out", c_void_p), ("ld_out", c_i64),
+        ("in_dtype", C.c_int32), ("nseq", C.c_int32), ("H", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
+        ("silu", C.c_int32), ("q_scale", c_float),
+    ]
+
+
+class MoeRouteParams(C.Structure):
+    _fields_ = [
+        ("x", c_void_p), ("ldx", c_i64), ("w", c_void_p), ("correction", c_void_p), ("gate_w", c_void_p),
+        ("idx", c_void_p), ("weight", c_void_p), ("gate", c_void_p),
+        ("x_dtype", C.c_int32), ("rows", C.c_int32), ("cols", C.c_int32), ("experts", C.c_int32), ("top", C.c_int32),
+        ("groups", C.c_int32), ("keep", C.c_int32), ("score", C.c_int32), ("group_top", C.c_int32), ("scale", c_float),
+    ]
+
+
+class TanhResidualParams(C.Structure):
+    _fields_ = [
+        ("x", c_void_p), ("table", c_void_p), ("ids", c_void_p),
+        ("a", c_void_p), ("b", c_void_p), ("part", c_void_p), ("h", c_void_p),
+        ("lda", c_i64), ("ldb", c_i64), ("ldp", c_i64), ("ldh", c_i64),
+        ("a_scale", c_void_p), ("b_scale", c_void_p), ("b_gate", c_void_p), ("idx", c_void_p), ("weight", c_void_p),
+        ("w", c_void_p * 2), ("bias", c_void_p * 2), ("out", c_void_p * 2), ("alpha", c_float * 2), ("mult", c_float),
+        ("table_dtype", C.c_int32), ("a_dtype", C.c_int32), ("b_dtype", C.c_int32), ("part_dtype", C.c_int32),
+        ("h_dtype", C.c_int32), ("out_dtype", C.c_int32), ("rows", C.c_int32), ("cols", C.c_int32),
+        ("n_partials", C.c_int32), ("experts", C.c_int32), ("n_out", C.c_int32),
     ]
 
 
@@ -297,6 +330,11 @@ SIGNATURES = {
     "vila_ssd_scan": [C.POINTER(SsdScanParams), c_void_p],
     "vila_delta_scan": [C.POINTER(DeltaScanParams), c_void_p],
     "vila_gla_scan": [C.POINTER(GlaScanParams), c_void_p],
+    "vila_decay_scan": [C.POINTER(DecayScanParams), c_void_p],
+    "vila_moe_route_scores": [C.POINTER(MoeRouteParams), c_void_p],
+    "vila_tanh_residual_rows": [C.POINTER(TanhResidualParams), c_void_p],
+    "vila_gated_head_norm_act_rows": [c_void_p, c_void_p, c_void_p, c_int, c_i64, c_float, c_void_p, c_int, c_int, c_int,
+                                      c_int, c_int, c_void_p],
     "vila_gated_head_norm_rows": [c_void_p, c_void_p, c_void_p, c_int, c_i64, c_float, c_void_p, c_int, c_int, c_int,
                                   c_int, c_void_p],
     "vila_scaled_residual_norm_rows": [c_void_p, c_void_p, c_int, c_i64, c_void_p, c_void_p, c_int, c_i64, c_void_p,

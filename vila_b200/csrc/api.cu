@@ -82,6 +82,10 @@ int vila_linear_act(const void* x, int64_t ldx, const void* w, int64_t ldw, cons
   vb::GemmEpilogue e = make_epi(bias, nullptr, 0, 0, act, flags);
   e.act_pos = act_pos;
   e.act_neg = act_neg;
+  if (flags & VILA_FLAG_GEGLU) {
+    VB_CHECK(act == VILA_ACT_NONE, "vila_linear_act: a gated unit takes no other activation (act=%d)", act);
+    e.swiglu = 3;
+  }
   if (flags & VILA_FLAG_GLU_CLAMP) {
     VB_CHECK(act == VILA_ACT_NONE, "vila_linear_act: the clamped gated unit takes no other activation (act=%d)", act);
     e.swiglu = 2;
@@ -459,8 +463,13 @@ int vila_moe_route_sigmoid(const void* x, int x_dtype, int64_t ldx, const float*
                            const float* correction, int32_t* idx, float* weight, int rows, int cols,
                            int experts, int top, int groups, int keep, void* stream) {
   VB_REQUIRE_DEVICE();
-  return vb::moe_route_sigmoid(x, x_dtype, ldx, w_router, correction, idx, weight, rows, cols, experts, top,
-                               groups, keep, st(stream));
+  vila_moe_route_params p = {};
+  p.x = x; p.x_dtype = x_dtype; p.ldx = ldx;
+  p.w = w_router; p.correction = correction;
+  p.idx = idx; p.weight = weight;
+  p.rows = rows; p.cols = cols; p.experts = experts; p.top = top; p.groups = groups; p.keep = keep;
+  p.score = VILA_SCORE_SIGMOID; p.group_top = 2; p.scale = 1.0f;
+  return vb::moe_route_scores(p, st(stream));
 }
 
 int vila_residual_norm_rows(float* x, const void* a, int a_dtype, int64_t lda, const void* part, int part_dtype,
@@ -541,6 +550,21 @@ int vila_gla_scan(const vila_gla_scan_params* p, void* stream) {
   return vb::gla_scan(*p, st(stream));
 }
 
+int vila_decay_scan(const vila_decay_scan_params* p, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::decay_scan(*p, st(stream));
+}
+
+int vila_moe_route_scores(const vila_moe_route_params* p, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::moe_route_scores(*p, st(stream));
+}
+
+int vila_tanh_residual_rows(const vila_tanh_residual_params* p, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::tanh_residual_rows(*p, st(stream));
+}
+
 int vila_scaled_residual_norm_rows(float* x, const void* a, int a_dtype, int64_t lda, const float* a_scale, const void* b,
                                    int b_dtype, int64_t ldb, const float* b_scale, const float* w, float eps, void* out,
                                    int out_dtype, int rows, int cols, void* stream) {
@@ -552,7 +576,13 @@ int vila_scaled_residual_norm_rows(float* x, const void* a, int a_dtype, int64_t
 int vila_gated_head_norm_rows(const float* o, const float* w, const void* gate, int gate_dtype, int64_t ldg, float eps,
                               void* out, int out_dtype, int rows, int H, int vdim, void* stream) {
   VB_REQUIRE_DEVICE();
-  return vb::gated_head_norm_rows(o, w, gate, gate_dtype, ldg, eps, out, out_dtype, rows, H, vdim, st(stream));
+  return vb::gated_head_norm_rows(o, w, gate, gate_dtype, ldg, eps, out, out_dtype, rows, H, vdim, VILA_ACT_SILU, st(stream));
+}
+
+int vila_gated_head_norm_act_rows(const float* o, const float* w, const void* gate, int gate_dtype, int64_t ldg, float eps,
+                                  void* out, int out_dtype, int rows, int H, int vdim, int gate_act, void* stream) {
+  VB_REQUIRE_DEVICE();
+  return vb::gated_head_norm_rows(o, w, gate, gate_dtype, ldg, eps, out, out_dtype, rows, H, vdim, gate_act, st(stream));
 }
 
 int vila_ssd_scan(const vila_ssd_scan_params* p, void* stream) {

@@ -439,12 +439,14 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         // every lane does useful SiLU work and one shuffle serves two tokens.
         const bool odd = (lane & 1) != 0;
         const uint32_t dst = smem_u32(buf) + ((n_local >> 1) + (odd ? 16 * (kStgPitch / 2) : 0)) * 2;
-        if (a.epi.swiglu == 2) {   // clamped gated unit on the unrounded accumulators
+        if (a.epi.swiglu >= 2) {   // clamped gated unit or gelu_tanh(gate) * up on the unrounded accumulators
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const float a0 = v[j] + bias, a1 = v[16 + j] + bias;
             const float recv = __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
-            sts_bf16(dst + j * kStgPitch, glu_clamp_fast_f(odd ? recv : a0, odd ? a1 : recv, a.epi.act_pos, a.epi.act_neg));
+            const float zg = odd ? recv : a0, zu = odd ? a1 : recv;
+            sts_bf16(dst + j * kStgPitch, a.epi.swiglu == 2 ? glu_clamp_fast_f(zg, zu, a.epi.act_pos, a.epi.act_neg)
+                                                            : gelu_tanh_f(zg) * zu);
           }
         } else {
 #pragma unroll

@@ -455,6 +455,18 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
             }
             continue;
           }
+          if (epi.swiglu == 3) {   // gelu_tanh(gate) * up, rounded once
+            if (row_ok) {
+              uint32_t o[8];
+#pragma unroll
+              for (int j = 0; j < 8; ++j)
+                o[j] = pack_bf16(gelu_tanh_f(v[4 * j + 0]) * v[4 * j + 1], gelu_tanh_f(v[4 * j + 2]) * v[4 * j + 3]);
+              __nv_bfloat16* dst = C + static_cast<size_t>(row) * ldc + (n0 >> 1);
+              if (n0 + 16 <= N) stg_v4(dst, make_uint4(o[0], o[1], o[2], o[3]));
+              if (n0 + 32 <= N) stg_v4(dst + 8, make_uint4(o[4], o[5], o[6], o[7]));
+            }
+            continue;
+          }
           if (epi.swiglu) {
             // interleaved (gate, up) column pairs -> 16 outputs: silu(gate) * up,
             // rounding to bf16 at the points the reference's unfused ops do.

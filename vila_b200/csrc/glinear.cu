@@ -24,6 +24,27 @@ __device__ __forceinline__ float glu_clamp_f(float zg, float zu, const vila_glin
   return g * sigmoid_f(x.act_alpha * g) * (u + 1.0f);
 }
 
+__device__ __forceinline__ float gelu_tanh_exact_f(float z) {
+  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float activate(float z, int act, const vila_glinear_ext& x) {
+  switch (act) {
+    case VILA_ACT_SILU: return silu_exact_f(z);
+    case VILA_ACT_RELU2: z = fmaxf(z, 0.f); return z * z;
+    case VILA_ACT_GELU_TANH: return gelu_tanh_exact_f(z);
+    case VILA_ACT_GELU_ERF: return gelu_erf_f(z);
+    case VILA_ACT_XIELU: return xielu_f(z, x.act_pos, x.act_neg);
+    case VILA_ACT_SOFTCAP: return x.act_pos * tanhf(z / x.act_pos);
+    default: return z;
+  }
+}
+// the two columns of a gated unit (flags: which one)
+constexpr int kGluFlags = VILA_FLAG_SWIGLU | VILA_FLAG_GLU_CLAMP | VILA_FLAG_GEGLU;
+__device__ __forceinline__ float glu(float g, float u, int flags, const vila_glinear_ext& x) {
+  if (flags & VILA_FLAG_GLU_CLAMP) return glu_clamp_f(g, u, x);
+  return (flags & VILA_FLAG_GEGLU ? gelu_tanh_exact_f(g) : silu_exact_f(g)) * u;
+}
+
 // scale of the INPUT row behind sorted position i (= output row: in_scale is only taken without o_rows)
 __device__ __forceinline__ float in_scale_of(const vila_glinear_params& p, const vila_glinear_ext& x, int i) {
   return x.in_scale ? x.in_scale[p.a_rows ? p.a_rows[i] : i] : 1.0f;
@@ -35,8 +56,7 @@ template <int TM>
 __device__ __forceinline__ void store_block(const vila_glinear_params& p, const vila_glinear_ext& x, int g, int n0,
                                             int tx, const int* orows, float (&acc)[TM][4]) {
   const size_t o_col0 = p.mode == 0 ? static_cast<size_t>(g) * p.o_group_off : 0;
-  const bool swiglu = (p.flags & VILA_FLAG_SWIGLU) != 0;
-  const bool glu_clamp = (p.flags & VILA_FLAG_GLU_CLAMP) != 0;
+  const bool gated = (p.flags & kGluFlags) != 0;
 #pragma unroll
   for (int i = 0; i < TM; ++i) {
     const int orow = orows[i];
@@ -49,25 +69,14 @@ __device__ __forceinline__ void store_block(const vila_glinear_params& p, const 
       const int n = n0 + tx * 4 + j;
       float z = acc[i][j] * is;
       if (p.bias && n < p.N) z += ld_any(p.bias, p.w_dtype, static_cast<size_t>(g) * p.bias_group_stride + n);
-      if (p.act == VILA_ACT_SILU) z = silu_exact_f(z);
-      else if (p.act == VILA_ACT_RELU2) { z = fmaxf(z, 0.f); z = z * z; }
-      else if (p.act == VILA_ACT_GELU_TANH) {
-        z = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-      } else if (p.act == VILA_ACT_XIELU) z = xielu_f(z, x.act_pos, x.act_neg);
-      v[j] = z;
+      v[j] = activate(z, p.act, x);
     }
     const size_t ob = static_cast<size_t>(orow) * p.ldo + o_col0;
-    if (glu_clamp) {
+    if (gated) {
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int n = n0 + tx * 4 + 2 * j;
-        if (n + 1 < p.N) st_any(p.out, p.out_dtype, ob + n / 2, glu_clamp_f(v[2 * j], v[2 * j + 1], x) * rs);
-      }
-    } else if (swiglu) {
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int n = n0 + tx * 4 + 2 * j;
-        if (n + 1 < p.N) st_any(p.out, p.out_dtype, ob + n / 2, silu_exact_f(v[2 * j]) * v[2 * j + 1] * rs);
+        if (n + 1 < p.N) st_any(p.out, p.out_dtype, ob + n / 2, glu(v[2 * j], v[2 * j + 1], p.flags, x) * rs);
       }
     } else {
 #pragma unroll
@@ -269,12 +278,7 @@ __device__ __forceinline__ void load8(const void* p, int dt, size_t i, float (&v
 
 __device__ __forceinline__ float finish(const vila_glinear_params& p, const vila_glinear_ext& x, float z, int g, int n) {
   if (p.bias) z += ld_any(p.bias, p.w_dtype, static_cast<size_t>(g) * p.bias_group_stride + n);
-  if (p.act == VILA_ACT_SILU) z = silu_exact_f(z);
-  else if (p.act == VILA_ACT_RELU2) { z = fmaxf(z, 0.f); z = z * z; }
-  else if (p.act == VILA_ACT_GELU_TANH)
-    z = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-  else if (p.act == VILA_ACT_XIELU) z = xielu_f(z, x.act_pos, x.act_neg);
-  return z;
+  return activate(z, p.act, x);
 }
 
 // vec: K % 8 == 0 and every row of A and W starts on an 8-element boundary (16 B bf16, 32 B fp32)
@@ -289,8 +293,7 @@ __global__ void __launch_bounds__(kSmallWarps * 32) glinear_small_kernel(const v
   const size_t wa = static_cast<size_t>(g) * p.w_group_stride + static_cast<size_t>(n_a) * p.ldw;
   const size_t wb = wa + p.ldw;
   const bool has_a = n_a < p.N, has_b = n_b < p.N;
-  const bool swiglu = (p.flags & VILA_FLAG_SWIGLU) != 0;
-  const bool glu_clamp = (p.flags & VILA_FLAG_GLU_CLAMP) != 0;
+  const bool gated = (p.flags & kGluFlags) != 0;
   for (int m0 = m_begin; m0 < m_end; m0 += kSmallRows) {
     const int nr = min(kSmallRows, m_end - m0);
     __syncthreads();
@@ -351,10 +354,8 @@ __global__ void __launch_bounds__(kSmallWarps * 32) glinear_small_kernel(const v
         if (lane == 0 && has_a) {
           const float rs = p.row_scale ? p.row_scale[orow] : 1.0f;
           const size_t ob = static_cast<size_t>(orow) * p.ldo + o_col0;
-          if (glu_clamp) {
-            if (has_b) st_any(p.out, p.out_dtype, ob + n_a / 2, glu_clamp_f(finish(p, x, za, g, n_a), finish(p, x, zb, g, n_b), x) * rs);
-          } else if (swiglu) {
-            if (has_b) st_any(p.out, p.out_dtype, ob + n_a / 2, silu_exact_f(finish(p, x, za, g, n_a)) * finish(p, x, zb, g, n_b) * rs);
+          if (gated) {
+            if (has_b) st_any(p.out, p.out_dtype, ob + n_a / 2, glu(finish(p, x, za, g, n_a), finish(p, x, zb, g, n_b), p.flags, x) * rs);
           } else {
             st_any(p.out, p.out_dtype, ob + n_a, finish(p, x, za, g, n_a) * rs);
             if (has_b) st_any(p.out, p.out_dtype, ob + n_b, finish(p, x, zb, g, n_b) * rs);
@@ -374,8 +375,10 @@ int glinear(const vila_glinear_params& p, cudaStream_t stream, const vila_glinea
   if (p.M <= 0 || p.N <= 0) return 0;
   VB_CHECK(p.K > 0 && p.groups >= 1, "glinear: K=%d groups=%d", p.K, p.groups);
   VB_CHECK(p.mode == 0 || (p.mode == 1 && p.seg != nullptr), "glinear: mode %d needs seg", p.mode);
-  VB_CHECK(!(p.flags & (VILA_FLAG_SWIGLU | VILA_FLAG_GLU_CLAMP)) || (p.N % 2 == 0 && p.act == VILA_ACT_NONE),
-           "glinear: the SwiGLU epilogue needs an even N and no other activation");
+  VB_CHECK(!(p.flags & kGluFlags) || (p.N % 2 == 0 && p.act == VILA_ACT_NONE),
+           "glinear: the epilogue of a gated unit needs an even N and no other activation");
+  VB_CHECK(p.act >= VILA_ACT_NONE && p.act <= VILA_ACT_SOFTCAP && (p.act != VILA_ACT_SOFTCAP || x.act_pos > 0.f),
+           "glinear: act=%d (cap %f)", p.act, x.act_pos);
   VB_CHECK(p.a_rows == nullptr || p.a_row_div >= 1, "glinear: a_row_div=%d", p.a_row_div);
   const bool small = p.M <= 16;
   // few rows: stream the weights once per 16-row chunk instead of tiling

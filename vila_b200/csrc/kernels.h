@@ -17,7 +17,7 @@ struct GemmEpilogue {
   int act = ACT_NONE;
   float act_pos = 0.f, act_neg = 0.f;  // ACT_XIELU: z > 0: act_pos z^2 + z / 2, else act_neg (e^z - 1 - z) + z / 2
   int swiglu = 0;  // interleaved (gate, up) columns -> N/2 outputs; 1: silu(gate) * up, 2: clamped gated unit with
-                   // alpha = act_pos, limit = act_neg
+                   // alpha = act_pos, limit = act_neg, 3: gelu_tanh(gate) * up
   int static_w = 0;  // W is a parameter: its first pipeline stages may be fetched before the PDL wait
   // split-K (set by the launcher): fp32 partial-sum workspace [M, N] (zeroed, self-cleaning) and
   // per-tile arrival counters (zeroed, self-cleaning)
@@ -235,7 +235,7 @@ int scaled_residual_norm_rows(float* x, const void* a, int a_dt, int64_t lda, co
                               int64_t ldb, const float* sb, const float* w, float eps, void* out, int o_dt, int rows,
                               int cols, cudaStream_t stream);
 int gated_head_norm_rows(const float* o, const float* w, const void* gate, int g_dt, int64_t ldg, float eps, void* out,
-                         int o_dt, int rows, int H, int vdim, cudaStream_t stream);
+                         int o_dt, int rows, int H, int vdim, int gate_act, cudaStream_t stream);
 int gated_norm_residual(float* x, const void* part, int p_dt, int64_t ldp, int np, const void* gate,
                         int g_dt, int64_t ldg, const void* gb, int b_dt, const void* w, int w_dt,
                         float w_off, float eps, int rows, int cols, cudaStream_t stream, float mult = 1.0f);
@@ -249,9 +249,6 @@ int residual_norm_rows(float* x, const void* a, int a_dt, int64_t lda, const voi
                        const void* w, int w_dt, float eps, void* out, int o_dt, int rows, int cols, cudaStream_t stream);
 int gelu_mul_gather(const void* z, int z_dt, const void* table, int dt, int64_t ldt, const int32_t* ids, int col0,
                     void* out, int o_dt, int rows, int cols, cudaStream_t stream);
-int moe_route_sigmoid(const void* x, int x_dt, int64_t ldx, const float* wr, const float* corr, int32_t* idx,
-                      float* weight, int rows, int cols, int experts, int top, int groups, int keep,
-                      cudaStream_t stream);
 int short_conv_rows(const float* h, const void* w, int w_dt, const float* state, const int32_t* seqs,
                     const int32_t* row_seq, void* out, int o_dt, int rows, int cols, int taps,
                     cudaStream_t stream);
@@ -281,12 +278,18 @@ struct vila_ssd_scan_params;
 struct vila_selective_scan_params;
 struct vila_delta_scan_params;
 struct vila_gla_scan_params;
+struct vila_decay_scan_params;
+struct vila_moe_route_params;
+struct vila_tanh_residual_params;
 namespace vb {
 int causal_conv_rows(const vila_causal_conv_params& p, cudaStream_t stream);
 int causal_conv_state(const vila_causal_conv_params& p, cudaStream_t stream);
 int causal_conv_step(const vila_causal_conv_params& p, cudaStream_t stream);
 int delta_scan(const vila_delta_scan_params& p, cudaStream_t stream);
 int gla_scan(const vila_gla_scan_params& p, cudaStream_t stream);
+int moe_route_scores(const vila_moe_route_params& p, cudaStream_t stream);
+int tanh_residual_rows(const vila_tanh_residual_params& p, cudaStream_t stream);
+int decay_scan(const vila_decay_scan_params& p, cudaStream_t stream);
 int ssd_scan(const vila_ssd_scan_params& p, cudaStream_t stream);
 int selective_scan(const vila_selective_scan_params& p, cudaStream_t stream);
 int norm_conv_rows(const vila_norm_conv_params& p, cudaStream_t stream);

@@ -7,11 +7,14 @@
 //                beta = sigmoid(b); head h uses q / k head h / (H / G)
 //   gla_scan     gated linear attention, one decay per key channel and token:
 //                  S <- diag(alpha) S + k v^T;  o = S^T (q_scale q),   alpha = sigmoid(z + z_bias)^(1 / tau)
+//   decay_scan   linear attention with one constant decay per head (lightning attention):
+//                  S <- g S + k v^T;  o = S^T (q_scale q);  optionally SiLU on q, k and v as they are read
 //
-// Both read-outs are taken from the state BEFORE the token's write, which is the same number and shortens the chain
+// The read-outs are taken from the state BEFORE the token's write, which is the same number and shortens the chain
 // of dependent steps to one pass over the state per token:
 //   delta:  S_new^T q = g (S^T q) + (k . q) u        so S^T k and S^T q are reduced together
 //   gla:    S_new^T q = S^T (alpha q) + (k . q) v    so the state update does not wait for the reduction
+//   decay:  S_new^T q = g (S^T q) + (k . q) v        likewise
 //
 // Grid (sequence, head, COLS columns of vdim).  Warps 0-3 own the state: R lanes share CPT columns, lane r
 // keeps the float4 pieces r, r + R, .. of a column in registers (state layout [.., vdim, dim]: coalesced loads, and
@@ -58,6 +61,9 @@ __device__ __forceinline__ float4 raw4_to_float(uint4 u, int dt) {
   return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
                      __uint_as_float(u.y & 0xffff0000u));
 }
+__device__ __forceinline__ float4 silu4(float4 v) {
+  return make_float4(silu_exact_f(v.x), silu_exact_f(v.y), silu_exact_f(v.z), silu_exact_f(v.w));
+}
 __device__ __forceinline__ float dot4(float4 a, float4 b, float s) {
   s = fmaf(a.x, b.x, s);
   s = fmaf(a.y, b.y, s);
@@ -89,6 +95,8 @@ __device__ __forceinline__ void transpose_sum(float (&v)[NV], int r) {
   }
 }
 
+enum Mode : int { kDelta, kGla, kDecay };
+
 struct ScanArgs {
   const void *q, *k, *v;        // rows of the step; head offsets are added by the kernel
   int64_t ldq, ldk, ldv;
@@ -101,18 +109,21 @@ struct ScanArgs {
   int64_t ldo;
   int in_dt, a_dt, H, G, dim, vdim;
   float q_scale, eps, inv_tau;
+  const float* decay;           // decay: [H]
+  int silu;                     // decay: q, k and v are pre-activations, SiLU is taken as they are read
   int vec_qk, vec_a;            // four-element loads of q | k and of z are aligned
 };
 
-template <bool DELTA, int R, int KPT, int CPT, int kStageWarps>
+template <int MODE, int R, int KPT, int CPT, int kStageWarps>
 __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_kernel(const ScanArgs p) {
   extern __shared__ __align__(16) float sm[];
+  constexpr bool DELTA = MODE == kDelta, GLA = MODE == kGla;
   constexpr int NP = R * KPT;                       // key channels the owners cover
   constexpr int NQ = KPT / 4;                       // float4 pieces per lane
   constexpr int GPW = 32 / R;                       // column groups per warp
   constexpr int COLS = kOwnerWarps * GPW * CPT;
   constexpr int NV = DELTA ? 2 * CPT : CPT;
-  constexpr int NVEC = DELTA ? 2 : 3;               // staged vectors per token: k, q (, alpha)
+  constexpr int NVEC = GLA ? 3 : 2;                 // staged vectors per token: k, q (, alpha)
   constexpr int TOK = NVEC * NP;
   constexpr int NG = NP > 128 ? NP / 128 : 1;       // four-element pieces a staging lane handles per vector
   constexpr int TPW = kChunk / kStageWarps;         // tokens of a stage per staging warp
@@ -140,7 +151,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
 #pragma unroll
     for (int j = 0; j < NG; ++j) {
       zb[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!DELTA && p.bias) {
+      if (GLA && p.bias) {
         const int i = 4 * (lane + 32 * j);
         float e[4];
 #pragma unroll
@@ -175,7 +186,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
             const int i = t < nt ? 4 * (lane + 32 * j) : dim;
             rk[u][j] = ld_raw4(p.k, dt, row * p.ldk + qoff, i, dim, p.vec_qk != 0);
             rq[u][j] = ld_raw4(p.q, dt, row * p.ldq + qoff, i, dim, p.vec_qk != 0);
-            if (!DELTA) rz[u][j] = ld_raw4(p.a, adt, row * p.lda + zoff, i, dim, p.vec_a != 0);
+            if (GLA) rz[u][j] = ld_raw4(p.a, adt, row * p.lda + zoff, i, dim, p.vec_a != 0);
           }
         }
 #pragma unroll
@@ -188,6 +199,10 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
           for (int j = 0; j < NG; ++j) {
             kv[j] = raw4_to_float(rk[u][j], dt);
             qv[j] = raw4_to_float(rq[u][j], dt);
+            if (MODE == kDecay && p.silu) {
+              kv[j] = silu4(kv[j]);
+              qv[j] = silu4(qv[j]);
+            }
             kq = dot4(kv[j], qv[j], kq);
             if (DELTA) {
               kk = dot4(kv[j], kv[j], kk);
@@ -211,7 +226,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
             if (i < NP) {
               float4 q4 = make_float4(qv[j].x * qs, qv[j].y * qs, qv[j].z * qs, qv[j].w * qs);
               *reinterpret_cast<float4*>(kd + i) = make_float4(kv[j].x * ks, kv[j].y * ks, kv[j].z * ks, kv[j].w * ks);
-              if (!DELTA) {
+              if (GLA) {
                 const float4 z = raw4_to_float(rz[u][j], adt);
                 const float4 al = make_float4(expf(-softplus_f(-(z.x + zb[j].x)) * p.inv_tau),
                                               expf(-softplus_f(-(z.y + zb[j].y)) * p.inv_tau),
@@ -229,7 +244,8 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
 #pragma unroll
       for (int k = 0; k < VN; ++k) {
         const int idx = st + k * kStageWarps * 32;
-        if (idx < kChunk * COLS) v_s[bf * kChunk * COLS + idx] = raw_to_float(rv[k], dt);
+        const float v = raw_to_float(rv[k], dt);
+        if (idx < kChunk * COLS) v_s[bf * kChunk * COLS + idx] = MODE == kDecay && p.silu ? silu_exact_f(v) : v;
       }
       if (DELTA && st < nt) {
         float* s = reinterpret_cast<float*>(sc_s + bf * kChunk + st);
@@ -282,6 +298,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
   const int mine = r / kSpan;                      // which of the NV sums this lane ends up with
   const int my_col = DELTA ? mine - CPT : mine;    // its column, if it is a read-out
   const bool writes = my_col >= 0 && (r % kSpan) == 0;
+  const float gh = MODE == kDecay ? p.decay[h] : 0.f;
   __syncthreads();
   for (int ch = 0; ch < nchunks; ++ch) {
     const int nt = min(kChunk, n - ch * kChunk), bf = ch & 1;
@@ -294,7 +311,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
     for (int j = 0; j < NQ; ++j) {
       kn[j] = reinterpret_cast<const float4*>(tok)[r + R * j];
       qn[j] = reinterpret_cast<const float4*>(tok + NP)[r + R * j];
-      if (!DELTA) an[j] = reinterpret_cast<const float4*>(tok + 2 * NP)[r + R * j];
+      if (GLA) an[j] = reinterpret_cast<const float4*>(tok + 2 * NP)[r + R * j];
     }
     for (int t = 0; t < nt; ++t) {
       float4 kc[NQ], qc[NQ], ac[NQ];
@@ -306,7 +323,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
       for (int j = 0; j < NQ; ++j) {
         kc[j] = kn[j];
         qc[j] = qn[j];
-        if (!DELTA) ac[j] = an[j];
+        if (GLA) ac[j] = an[j];
       }
       // the next token's vectors (row kChunk of a buffer does not exist: the last token reads its own again)
       const float* nx = tok + (t + 1 < nt ? t + 1 : t) * TOK;
@@ -314,7 +331,7 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
       for (int j = 0; j < NQ; ++j) {
         kn[j] = reinterpret_cast<const float4*>(nx)[r + R * j];
         qn[j] = reinterpret_cast<const float4*>(nx + NP)[r + R * j];
-        if (!DELTA) an[j] = reinterpret_cast<const float4*>(nx + 2 * NP)[r + R * j];
+        if (GLA) an[j] = reinterpret_cast<const float4*>(nx + 2 * NP)[r + R * j];
       }
       float d[NV];
 #pragma unroll
@@ -359,13 +376,13 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
           if (c == my_col) vm = vc[c];
 #pragma unroll
           for (int j = 0; j < NQ; ++j) {
-            S[c][j].x = fmaf(ac[j].x, S[c][j].x, kc[j].x * vc[c]);
-            S[c][j].y = fmaf(ac[j].y, S[c][j].y, kc[j].y * vc[c]);
-            S[c][j].z = fmaf(ac[j].z, S[c][j].z, kc[j].z * vc[c]);
-            S[c][j].w = fmaf(ac[j].w, S[c][j].w, kc[j].w * vc[c]);
+            S[c][j].x = fmaf(GLA ? ac[j].x : gh, S[c][j].x, kc[j].x * vc[c]);
+            S[c][j].y = fmaf(GLA ? ac[j].y : gh, S[c][j].y, kc[j].y * vc[c]);
+            S[c][j].z = fmaf(GLA ? ac[j].z : gh, S[c][j].z, kc[j].z * vc[c]);
+            S[c][j].w = fmaf(GLA ? ac[j].w : gh, S[c][j].w, kc[j].w * vc[c]);
           }
         }
-        if (writes) yy[t * COLS + cg + my_col] = fmaf(s4.z, vm, d[0]);
+        if (writes) yy[t * COLS + cg + my_col] = fmaf(s4.z, vm, GLA ? d[0] : gh * d[0]);
       }
     }
     __syncthreads();
@@ -388,15 +405,15 @@ __global__ void __launch_bounds__(32 * (kOwnerWarps + kStageWarps)) outer_scan_k
     }
 }
 
-template <bool DELTA, int R, int KPT, int CPT>
+template <int MODE, int R, int KPT, int CPT>
 int launch_scan(const ScanArgs& p, int nseq, cudaStream_t stream) {
   constexpr int NP = R * KPT, COLS = kOwnerWarps * (32 / R) * CPT;
-  constexpr size_t smem = sizeof(float) * (2 * kChunk * (DELTA ? 2 : 3) * NP + 4 * kChunk * COLS + 2 * kChunk * 4);
+  constexpr size_t smem = sizeof(float) * (2 * kChunk * (MODE == kGla ? 3 : 2) * NP + 4 * kChunk * COLS + 2 * kChunk * 4);
   static_assert(smem <= 224 * 1024, "outer_scan: shared memory");
   // the staging work of a token is the same for 2 as for 4 columns per group: twice the warps for the narrow form,
   // where an SM holds one or two CTAs, fewer for the wide one, where CTAs share it
   constexpr int SW = CPT == 4 ? 4 : 8;
-  auto kern = outer_scan_kernel<DELTA, R, KPT, CPT, SW>;
+  auto kern = outer_scan_kernel<MODE, R, KPT, CPT, SW>;
   static PerDeviceOnce attr_once;
   if (smem > 48 * 1024 && attr_once.first())
     VB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
@@ -408,20 +425,20 @@ int launch_scan(const ScanArgs& p, int nseq, cudaStream_t stream) {
 
 // columns per lane group: four where the launch still fills the machine twice over, else fewer, so that one long
 // prompt spreads over more CTAs
-template <bool DELTA, int R, int KPT>
+template <int MODE, int R, int KPT>
 int pick_columns(const ScanArgs& p, int nseq, cudaStream_t stream) {
   const long groups = static_cast<long>(nseq) * p.H * ((p.vdim + 4 * (32 / R) - 1) / (4 * (32 / R)));   // CTAs at CPT = 1
-  if (groups >= 8L * num_sms()) return launch_scan<DELTA, R, KPT, 4>(p, nseq, stream);
-  return launch_scan<DELTA, R, KPT, 2>(p, nseq, stream);
+  if (groups >= 8L * num_sms()) return launch_scan<MODE, R, KPT, 4>(p, nseq, stream);
+  return launch_scan<MODE, R, KPT, 2>(p, nseq, stream);
 }
 
-template <bool DELTA>
+template <int MODE>
 int scan_by_dim(const ScanArgs& p, int nseq, cudaStream_t stream) {
-  if (p.dim <= 32) return pick_columns<DELTA, 8, 4>(p, nseq, stream);
-  if (p.dim <= 64) return pick_columns<DELTA, 16, 4>(p, nseq, stream);
-  if (p.dim <= 128) return pick_columns<DELTA, 16, 8>(p, nseq, stream);
-  if (p.dim <= 256) return pick_columns<DELTA, 16, 16>(p, nseq, stream);
-  return pick_columns<DELTA, 32, 16>(p, nseq, stream);
+  if (p.dim <= 32) return pick_columns<MODE, 8, 4>(p, nseq, stream);
+  if (p.dim <= 64) return pick_columns<MODE, 16, 4>(p, nseq, stream);
+  if (p.dim <= 128) return pick_columns<MODE, 16, 8>(p, nseq, stream);
+  if (p.dim <= 256) return pick_columns<MODE, 16, 16>(p, nseq, stream);
+  return pick_columns<MODE, 32, 16>(p, nseq, stream);
 }
 
 // rows that start on a four-element boundary of their dtype (8 bytes bf16, 16 bytes fp32)
@@ -450,7 +467,7 @@ int delta_scan(const vila_delta_scan_params& p, cudaStream_t stream) {
   a.H = p.H; a.G = p.G; a.dim = p.dim; a.vdim = p.vdim;
   a.q_scale = p.q_scale; a.eps = p.unit_eps;
   a.vec_qk = p.dim % 4 == 0 && rows_aligned4(a.q, p.ld_qkv, p.in_dtype) && rows_aligned4(a.k, p.ld_qkv, p.in_dtype);
-  return scan_by_dim<true>(a, p.nseq, stream);
+  return scan_by_dim<kDelta>(a, p.nseq, stream);
 }
 
 int gla_scan(const vila_gla_scan_params& p, cudaStream_t stream) {
@@ -468,7 +485,24 @@ int gla_scan(const vila_gla_scan_params& p, cudaStream_t stream) {
   a.q_scale = p.q_scale; a.inv_tau = 1.0f / p.tau;
   a.vec_qk = p.dim % 4 == 0 && rows_aligned4(a.q, p.ld_q, p.in_dtype) && rows_aligned4(a.k, p.ld_k, p.in_dtype);
   a.vec_a = p.dim % 4 == 0 && rows_aligned4(a.a, p.ld_z, p.z_dtype);
-  return scan_by_dim<false>(a, p.nseq, stream);
+  return scan_by_dim<kGla>(a, p.nseq, stream);
+}
+
+int decay_scan(const vila_decay_scan_params& p, cudaStream_t stream) {
+  if (p.nseq <= 0) return 0;
+  VB_CHECK(p.H >= 1 && p.dim >= 1 && p.dim <= 512 && p.vdim >= 1 && p.decay != nullptr, "decay_scan: H=%d dim=%d (<= 512) vdim=%d",
+           p.H, p.dim, p.vdim);
+  ScanArgs a = {};
+  a.q = p.q; a.k = p.k; a.v = p.v;
+  a.ldq = p.ld_q; a.ldk = p.ld_k; a.ldv = p.ld_v;
+  a.decay = p.decay;
+  a.silu = p.silu;
+  a.state = p.state; a.seqs = p.seqs; a.out = p.out; a.ldo = p.ld_out;
+  a.in_dt = p.in_dtype;
+  a.H = p.H; a.G = p.H; a.dim = p.dim; a.vdim = p.vdim;
+  a.q_scale = p.q_scale;
+  a.vec_qk = p.dim % 4 == 0 && rows_aligned4(a.q, p.ld_q, p.in_dtype) && rows_aligned4(a.k, p.ld_k, p.in_dtype);
+  return scan_by_dim<kDecay>(a, p.nseq, stream);
 }
 
 }  // namespace vb

@@ -26,6 +26,10 @@
 // weights exp(s - max) / sum, mixed over heads, times the values (pass 1; nothing is rescaled).  When the keys of
 // a decoded token are dealt to several CTAs, pass 0 and pass 1 are two launches: the first leaves every CTA's
 // (max, sum) of its share in the partial records, the second merges them in split order and adds its share.
+// Differential attention (maps == 2): every query / key head comes as two maps side by side, each an attention of its own
+// over the same value head; a CTA always holds both maps of its heads, so the pair is combined where the sums end,
+//   o = rms(a1 - lambda a2) * diff_scale   (rms over the head's vdim values), then the gate,
+// in the epilogue of the tiled and the one-row kernel or in the merge of a decoded token's key splits.
 // Every reduction over keys runs in key order inside a block and block by block, so a row's result does
 // not depend on what else is in the launch.
 #include "../../include/vila_b200.h"
@@ -45,6 +49,8 @@ __host__ __device__ __forceinline__ int round4(int r) { return (r + 3) & ~3; }
 // plus a pad that makes the stride 4 mod 32, so that the float4 reads of 8 consecutive keys (same head, same
 // column) fall into 8 different bank groups.
 __host__ __device__ __forceinline__ int key_stride(int G, int DS) { return G * DS + ((36 - (G * DS) % 32) % 32); }
+
+__host__ __device__ __forceinline__ int maps_of(int maps) { return maps > 1 ? maps : 1; }
 
 // ---- rotary + unit norm + append ---------------------------------------------------------------------
 // One CTA per token; warp w takes the heads w, w + 8, ... of q then k; v is copied by all threads.
@@ -67,9 +73,11 @@ __global__ void __launch_bounds__(kThreads) rope_append_kernel(const vila_rope_a
   auto pair_of = [&](int c) { return halves ? (c < half ? c : c - half) : (c >> 1); };
   auto second = [&](int c) { return halves ? c >= half : (c & 1) != 0; };
   const size_t in0 = static_cast<size_t>(t) * p.ldq;
-  const size_t prow = static_cast<size_t>(p.cache_rows[t]) * (static_cast<size_t>(p.G) * (p.dim + p.vdim));
-  for (int hh = warp; hh < p.H + p.G; hh += kWarps) {
-    const bool is_q = hh < p.H;
+  const int maps = maps_of(p.maps), HQ = p.H * maps, GK = p.G * maps;   // query / key heads with their maps counted singly
+  const size_t koff = static_cast<size_t>(GK) * p.dim;                  // where a pool row's values start
+  const size_t prow = static_cast<size_t>(p.cache_rows[t]) * (koff + static_cast<size_t>(p.G) * p.vdim);
+  for (int hh = warp; hh < HQ + GK; hh += kWarps) {
+    const bool is_q = hh < HQ;
     const size_t src = in0 + static_cast<size_t>(hh) * p.dim;   // q heads then k heads are contiguous
     // pass 1: rotated values -> sum of squares (recomputed in pass 2: dim is small, no buffer needed)
     float ss = 0.f;
@@ -88,7 +96,7 @@ __global__ void __launch_bounds__(kThreads) rope_append_kernel(const vila_rope_a
     for (int c = lane; c < p.dim; c += 32) {
       float v = ld_any(p.qkv, p.qkv_dtype, src + c);
       if (p.v_from_k && !is_q)   // the value is the key as it came in
-        st_any(p.pool, p.pool_dtype, prow + static_cast<size_t>(p.G) * p.dim + static_cast<size_t>(hh - p.H) * p.dim + c, v);
+        st_any(p.pool, p.pool_dtype, prow + koff + static_cast<size_t>(hh - HQ) * p.dim + c, v);
       if (c < p.rot_dims) {
         const float o = ld_any(p.qkv, p.qkv_dtype, src + partner(c));
         const float co = cs[pair_of(c)], si = cs[half + pair_of(c)];
@@ -96,12 +104,12 @@ __global__ void __launch_bounds__(kThreads) rope_append_kernel(const vila_rope_a
       }
       v *= r;
       if (nw) v *= nw[c];
-      if (is_q) p.q_out[(static_cast<size_t>(t) * p.H + hh) * p.dim + c] = v;
-      else st_any(p.pool, p.pool_dtype, prow + static_cast<size_t>(hh - p.H) * p.dim + c, v);
+      if (is_q) p.q_out[(static_cast<size_t>(t) * HQ + hh) * p.dim + c] = v;
+      else st_any(p.pool, p.pool_dtype, prow + static_cast<size_t>(hh - HQ) * p.dim + c, v);
     }
   }
   if (p.v_from_k) return;
-  const size_t vsrc = in0 + static_cast<size_t>(p.H + p.G) * p.dim, vdst = prow + static_cast<size_t>(p.G) * p.dim;
+  const size_t vsrc = in0 + static_cast<size_t>(HQ + GK) * p.dim, vdst = prow + koff;
   for (int c = tid; c < p.G * p.vdim; c += kThreads) {
     float v = ld_any(p.qkv, p.qkv_dtype, vsrc + c);
     if (p.v_first)   // part of the value comes from another layer's value of the same token
@@ -115,8 +123,8 @@ struct AttnShape {
   int BQ;      // query rows per CTA
   int BK;      // keys per block (<= 32: one lane per key in the softmax step)
   int sub;     // CTAs per 16-row tile (grid.y)
-  int hsplit;  // head groups per tile (grid.z of the tiled kernel): 1 = all heads in one CTA, G = one K/V head and
-               // its query heads per CTA (possible when the heads' scores are not mixed)
+  int hsplit;  // head groups per tile (grid.z of the tiled kernel, inside grid.y of the other): 1 = all heads in one
+               // CTA, G = one K/V head and its query heads per CTA (possible when the heads' scores are not mixed)
   int phase;   // weights mixed after the softmax with the keys of a row dealt to several CTAs: 0 = this launch only
                // leaves every CTA's running (max, sum) in its partial record, 1 = this launch merges those records and
                // adds its share of the values; -1 = one CTA does both passes itself
@@ -162,21 +170,28 @@ __device__ __forceinline__ float capped(const vila_paged_attn_params& p, float s
 __device__ __forceinline__ float dist_bias(const vila_paged_attn_params& p, int dist, int h) {
   return __ldg(p.dist_bias + static_cast<size_t>(min(dist, p.dist_rows - 1)) * p.H + h);
 }
+// Score head h counts the maps singly: model head h / maps, map h % maps.  Its key head (also counted with maps) and
+// value head; rep = query heads per key / value head.
+__device__ __forceinline__ int key_head(int h, int maps, int rep) { return maps == 1 ? h / rep : ((h >> 1) / rep) * 2 + (h & 1); }
+__device__ __forceinline__ int value_head(int h, int maps, int rep) { return maps == 1 ? h / rep : (h >> 1) / rep; }
 __device__ __forceinline__ float out_gate(const vila_paged_attn_params& p, int row, int h) {
   return p.gate ? sigmoid_f(ld_any(p.gate, p.gate_dtype, static_cast<size_t>(row) * p.ldg + h)) : 1.0f;
 }
 
 // K | V rows of a key block, widened to fp32: one warp per key.  16-byte loads when the head sizes allow
 // (bf16: multiples of 8, fp32: multiples of 4; the pool row is then 16-byte aligned as well).
-// g0, G: the K/V heads g0 .. g0 + G - 1 of the pool row are loaded (all of them by default).
+// g0, G: the value heads g0 .. g0 + G - 1 of the pool row are loaded (all of them by default) with their key heads (as
+// many, or one per map).
 __device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_paged_attn_params& p,
                                               const int32_t* pt, int j0, int nkeys, int BK, int D4, int DS, int V4,
                                               int nwarps = kWarps, int g0 = 0, int G = 0, bool with_v = true) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (G == 0) G = p.G;
-  const int D = p.dim, V = p.vdim, KS = key_stride(G, DS);
-  const size_t prw = static_cast<size_t>(p.G) * (D + V);
-  const size_t koff = static_cast<size_t>(g0) * D, voff = static_cast<size_t>(p.G) * D + static_cast<size_t>(g0) * V;
+  const int maps = maps_of(p.maps), GK = G * maps;
+  const int D = p.dim, V = p.vdim, KS = key_stride(GK, DS);
+  const size_t prw = static_cast<size_t>(p.G) * (maps * D + V);
+  const size_t koff = static_cast<size_t>(g0) * maps * D;
+  const size_t voff = static_cast<size_t>(p.G) * maps * D + static_cast<size_t>(g0) * V;
   const bool vec16 = p.pool_dtype == VILA_DT_BF16 && (D & 7) == 0 && (V & 7) == 0;
   const bool vec32 = p.pool_dtype == VILA_DT_F32 && (D & 3) == 0 && (V & 3) == 0;
   for (int jj = warp; jj < BK; jj += nwarps) {
@@ -193,7 +208,7 @@ __device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_p
       const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.pool) + src;
       const uint4* k4 = reinterpret_cast<const uint4*>(base + koff);
       const uint4* v4 = reinterpret_cast<const uint4*>(base + voff);
-      for (int x = lane; x < (G * D) >> 3; x += 32) {
+      for (int x = lane; x < (GK * D) >> 3; x += 32) {
         const uint4 u = __ldg(k4 + x);
         const int e = x << 3, g = e / D, k = e - g * D;
         float* d = kd + g * DS + k;
@@ -214,13 +229,13 @@ __device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_p
       const float* base = static_cast<const float*>(p.pool) + src;
       const float4* k4 = reinterpret_cast<const float4*>(base + koff);
       const float4* v4 = reinterpret_cast<const float4*>(base + voff);
-      for (int x = lane; x < (G * D) >> 2; x += 32) {
+      for (int x = lane; x < (GK * D) >> 2; x += 32) {
         const int e = x << 2, g = e / D, k = e - g * D;
         *reinterpret_cast<float4*>(kd + g * DS + k) = __ldg(k4 + x);
       }
       for (int x = lane; with_v && x < (G * V) >> 2; x += 32) *reinterpret_cast<float4*>(vd + (x << 2)) = __ldg(v4 + x);
     } else {
-      for (int x = lane; x < G * D4; x += 32) {
+      for (int x = lane; x < GK * D4; x += 32) {
         const int g = x / D4, k = x - g * D4;
         kd[g * DS + k] = k < D ? ld_any(p.pool, p.pool_dtype, src + koff + static_cast<size_t>(g) * D + k) : 0.f;
       }
@@ -233,18 +248,37 @@ __device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_p
   }
 }
 
+// Differential attention: a warp turns the two maps' finished rows of one head (fp32 in shared memory, V values each)
+// into the head's output.
+__device__ __forceinline__ void combine_maps(const vila_paged_attn_params& p, const float* a1, const float* a2, int row, int h) {
+  const int lane = threadIdx.x & 31, V = p.vdim;
+  float ss = 0.f;
+  for (int c = lane; c < V; c += 32) {
+    const float o = fmaf(-p.diff_lambda, a2[c], a1[c]);
+    ss = fmaf(o, o, ss);
+  }
+  ss = warp_sum(ss);
+  const float r = p.diff_scale / sqrtf(ss / static_cast<float>(V) + p.diff_eps) * out_gate(p, row, h);
+  const size_t ob = (static_cast<size_t>(row) * p.H + h) * V;
+  for (int c = lane; c < V; c += 32) st_any(p.out, p.out_dtype, ob + c, fmaf(-p.diff_lambda, a2[c], a1[c]) * r);
+}
+
 // Shared memory (floats):  Qs [BQ * H][D4] (scale folded in) | Ks [BK][G][DS] | Vs [BK][G][V4] |
 //   Ss [BQ * H][BK] raw scores | Ps [BQ * H][BK] weights | talk [H * H] | m, l, alpha [BQ * H]
+// H and G count score heads (a head's maps singly), the value heads are GV = G / maps.
 // DS = D4 + 4: consecutive keys start 4 banks apart, so the float4 reads of 8 keys do not collide.
 template <int NACC>
 __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_attn_params p, const AttnShape sh) {
   extern __shared__ __align__(16) float sm[];
-  const int H = p.H, G = p.G, D = p.dim, V = p.vdim, BQ = sh.BQ, BK = sh.BK;
+  // H, G: the heads this CTA serves (all of them, or one value head with its key and query heads: h0 + h, g0 + g)
+  const int maps = maps_of(p.maps), HT = p.H * maps, hs = blockIdx.y % sh.hsplit;
+  const int H = HT / sh.hsplit, GV = p.G / sh.hsplit, G = GV * maps, h0 = hs * H, g0 = hs * GV;
+  const int D = p.dim, V = p.vdim, BQ = sh.BQ, BK = sh.BK;
   const int D4 = round4(D), DS = D4 + 4, V4 = round4(V), R = BQ * H, rep = H / G, KS = key_stride(G, DS);
   float* Qs = sm;
   float* Ks = Qs + R * D4;
   float* Vs = Ks + BK * KS;
-  float* Ss = Vs + BK * G * V4;
+  float* Ss = Vs + BK * GV * V4;
   float* Ps = Ss + R * BK;
   float* Tk = Ps + R * BK;
   float* m_s = Tk + H * H;
@@ -252,23 +286,22 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
   float* a_s = l_s + R;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int* tile = p.tiles + 4 * blockIdx.x;
-  const int i0 = blockIdx.y * BQ;
+  const int i0 = blockIdx.y / sh.hsplit * BQ;
   const int n_tile = tile[1];
   if (i0 >= n_tile) return;
   const int row0 = tile[0] + i0, n = min(BQ, n_tile - i0), pos0 = tile[2] + i0;
   const int32_t* pt = p.page_tables + static_cast<size_t>(tile[3]) * p.pt_stride;
   const int split = blockIdx.z, nsplit = gridDim.z;
-  const size_t prw = static_cast<size_t>(G) * (D + V);   // pool row width
 
   for (int idx = tid; idx < R * D4; idx += kThreads) {
     const int r = idx / D4, k = idx - r * D4, i = r / H, h = r - i * H;
-    Qs[idx] = (i < n && k < D) ? p.q[(static_cast<size_t>(row0 + i) * H + h) * D + k] * head_scale(p, h) : 0.f;
+    Qs[idx] = (i < n && k < D) ? p.q[(static_cast<size_t>(row0 + i) * HT + h0 + h) * D + k] * head_scale(p, h0 + h) : 0.f;
   }
   for (int idx = tid; idx < H * H; idx += kThreads) Tk[idx] = p.talk ? p.talk[idx] : ((idx / H) == (idx % H) ? 1.f : 0.f);
   const bool after = p.talk_after != 0 && p.talk != nullptr;
   for (int r = tid; r < R; r += kThreads) {
     const bool first = split == 0 && p.sink != nullptr && !after;
-    m_s[r] = first ? p.sink[r % H] : kNegBig;
+    m_s[r] = first ? p.sink[h0 + r % H] : kNegBig;
     l_s[r] = first ? 1.0f : 0.0f;
   }
   float4 acc[NACC];
@@ -304,13 +337,13 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
   for (int vb_ = all_blocks ? 0 : split; vb_ < bl.count; vb_ += all_blocks ? 1 : nsplit) {
     const int j0 = bl.block(vb_) * BK;
     __syncthreads();
-    load_kv_block(Ks, Vs, p, pt, j0, nkeys, BK, D4, DS, V4, kWarps, 0, 0, !stats);
+    load_kv_block(Ks, Vs, p, pt, j0, nkeys, BK, D4, DS, V4, kWarps, g0, GV, !stats);
     __syncthreads();
     // raw scores of every (score row, key)
     for (int idx = tid; idx < R * BK; idx += kThreads) {
       const int r = idx / BK, jj = idx - r * BK, h = r % H;
       const float4* qr = reinterpret_cast<const float4*>(Qs + r * D4);
-      const float4* kr = reinterpret_cast<const float4*>(Ks + jj * KS + (h / rep) * DS);
+      const float4* kr = reinterpret_cast<const float4*>(Ks + jj * KS + key_head(h, maps, rep) * DS);
       float s = 0.f;
 #pragma unroll 4
       for (int k = 0; k < (D4 >> 2); ++k) {
@@ -369,7 +402,7 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
           s = Ss[r * BK + lane];
         }
       }
-      if (valid && p.dist_bias) s += dist_bias(p, pos0 + i - (j0 + lane), h);
+      if (valid && p.dist_bias) s += dist_bias(p, pos0 + i - (j0 + lane), h0 + h);
       s = valid ? s : kNegBig;
       const float m_old = m_s[r];
       const float m_new = fmaxf(m_old, warp_max(s));
@@ -394,10 +427,10 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
         float4 v = acc[a];
         v.x *= alpha; v.y *= alpha; v.z *= alpha; v.w *= alpha;
         const float* pr = Ps + r * BK;
-        const float* vr = Vs + (h / rep) * V4 + 4 * c4;
+        const float* vr = Vs + value_head(h, maps, rep) * V4 + 4 * c4;
         for (int jj = 0; jj < BK; ++jj) {
           const float pj = pr[jj];
-          const float4 c = *reinterpret_cast<const float4*>(vr + jj * G * V4);
+          const float4 c = *reinterpret_cast<const float4*>(vr + jj * GV * V4);
           v.x = fmaf(pj, c.x, v.x); v.y = fmaf(pj, c.y, v.y); v.z = fmaf(pj, c.z, v.z); v.w = fmaf(pj, c.w, v.w);
         }
         acc[a] = v;
@@ -406,6 +439,30 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
   }
   }
   __syncthreads();
+  if (maps > 1 && nsplit == 1) {   // finished rows to shared memory (over the operands), then a warp per (row, head)
+#pragma unroll
+    for (int a = 0; a < NACC; ++a) {
+      const int o = tid + a * kThreads;
+      if (o < nout) {
+        const float inv = 1.0f / l_s[o / vq];
+        acc[a].x *= inv; acc[a].y *= inv; acc[a].z *= inv; acc[a].w *= inv;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int a = 0; a < NACC; ++a) {
+      const int o = tid + a * kThreads;
+      if (o < nout) *reinterpret_cast<float4*>(sm + 4 * o) = acc[a];   // [R][V4]
+    }
+    __syncthreads();
+    const int HM = H / maps;   // heads of this CTA
+    for (int u = warp; u < n * HM; u += kWarps) {
+      const int i = u / HM, h = u - i * HM;
+      const float* a1 = sm + (i * H + 2 * h) * V4;
+      combine_maps(p, a1, a1 + V4, row0 + i, h0 / maps + h);
+    }
+    return;
+  }
 #pragma unroll
   for (int a = 0; a < NACC; ++a) {
     const int o = tid + a * kThreads;
@@ -414,13 +471,13 @@ __global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_a
     if (i >= n) continue;
     const float v[4] = {acc[a].x, acc[a].y, acc[a].z, acc[a].w};
     if (nsplit == 1) {
-      const float inv = after ? out_gate(p, row0 + i, h) : out_gate(p, row0 + i, h) / l_s[r];
-      const size_t ob = (static_cast<size_t>(row0 + i) * H + h) * V + 4 * c4;
+      const float inv = after ? out_gate(p, row0 + i, h0 + h) : out_gate(p, row0 + i, h0 + h) / l_s[r];
+      const size_t ob = (static_cast<size_t>(row0 + i) * HT + h0 + h) * V + 4 * c4;
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if (4 * c4 + e < V) st_any(p.out, p.out_dtype, ob + e, v[e] * inv);
     } else {
-      float* part = p.partial + ((static_cast<size_t>(row0 + i) * nsplit + split) * H + h) * (V + 2);
+      float* part = p.partial + ((static_cast<size_t>(row0 + i) * nsplit + split) * HT + h0 + h) * (V + 2);
       if (!(after && sh.phase == 0)) {
 #pragma unroll
         for (int e = 0; e < 4; ++e)
@@ -445,13 +502,14 @@ template <int NACC, int NT, int TR>
 __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_attn_params p, const AttnShape sh) {
   extern __shared__ __align__(16) float sm[];
   // H, G: the heads this CTA serves (all of them, or one K/V head with its query heads: global heads h0 + h, g0 + g)
-  const int H = p.H / sh.hsplit, G = p.G / sh.hsplit, h0 = blockIdx.z * H, g0 = blockIdx.z * G;
+  const int maps = maps_of(p.maps), HT = p.H * maps;
+  const int H = HT / sh.hsplit, GV = p.G / sh.hsplit, G = GV * maps, h0 = blockIdx.z * H, g0 = blockIdx.z * GV;
   const int D = p.dim, V = p.vdim, BQ = sh.BQ, BK = sh.BK, HK = sh.BK >> 1;
   const int D4 = round4(D), DS = D4 + 4, V4 = round4(V), R = BQ * H, NB = R >> 2, rep = H / G, KS = key_stride(G, DS);
   float* Qs = sm;
   float* Ks = Qs + R * D4;
   float* Vs = Ks + BK * KS;
-  float* Ss = Vs + BK * G * V4;
+  float* Ss = Vs + BK * GV * V4;
   float* Ps = Ss + R * BK;
   float* m_s = Ps + R * BK;
   float* l_s = m_s + R;
@@ -467,7 +525,7 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
 
   for (int idx = tid; idx < R * D4; idx += NT) {
     const int r = idx / D4, k = idx - r * D4, h = r / BQ, i = r - h * BQ;
-    Qs[idx] = (i < n && k < D) ? p.q[(static_cast<size_t>(row0 + i) * p.H + h0 + h) * D + k] * head_scale(p, h0 + h) : 0.f;
+    Qs[idx] = (i < n && k < D) ? p.q[(static_cast<size_t>(row0 + i) * HT + h0 + h) * D + k] * head_scale(p, h0 + h) : 0.f;
   }
   for (int idx = tid; idx < H * H; idx += NT) Tk[idx] = p.talk ? p.talk[idx] : ((idx / H) == (idx % H) ? 1.f : 0.f);
   const bool after = p.talk_after != 0 && p.talk != nullptr;
@@ -496,11 +554,11 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
   for (int vb_ = 0; vb_ < bl.count; ++vb_) {
     const int j0 = bl.block(vb_) * BK;
     __syncthreads();
-    load_kv_block(Ks, Vs, p, pt, j0, nkeys, BK, D4, DS, V4, NT / 32, g0, G, !stats);
+    load_kv_block(Ks, Vs, p, pt, j0, nkeys, BK, D4, DS, V4, NT / 32, g0, GV, !stats);
     __syncthreads();
     for (int item = tid; item < (R / TR) * HK; item += NT) {
       const int rbs = item / HK, jp = item - rbs * HK, r0 = rbs * TR;     // TR score rows of one head x 2 keys
-      const int g = (r0 / BQ) / rep;
+      const int g = key_head(r0 / BQ, maps, rep);
       const float4* q0 = reinterpret_cast<const float4*>(Qs + r0 * D4);
       const float4* k0 = reinterpret_cast<const float4*>(Ks + jp * KS + g * DS);
       const float4* k1 = reinterpret_cast<const float4*>(Ks + (jp + HK) * KS + g * DS);
@@ -628,7 +686,7 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
       const int o = tid + a * NT;
       if (o < nout) {
         const int rb = o / vq, c4 = o - rb * vq;
-        const int g = ((rb << 2) / BQ) / rep;
+        const int g = value_head((rb << 2) / BQ, maps, rep);
         const float4 al = *reinterpret_cast<const float4*>(a_s + (rb << 2));
         const float alv[4] = {al.x, al.y, al.z, al.w};
 #pragma unroll
@@ -640,7 +698,7 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
 #pragma unroll 4
         for (int jj = 0; jj < BK; ++jj) {
           const float4 pw = pr[jj];
-          const float4 c = *reinterpret_cast<const float4*>(vr + jj * G * V4);
+          const float4 c = *reinterpret_cast<const float4*>(vr + jj * GV * V4);
           const float pv[4] = {pw.x, pw.y, pw.z, pw.w};
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
@@ -653,6 +711,38 @@ __global__ void __launch_bounds__(NT) paged_attn_tile4_kernel(const vila_paged_a
   }
   }
   __syncthreads();
+  if (maps > 1) {   // finished rows to shared memory (over the operands), then a warp per (row, head)
+#pragma unroll
+    for (int a = 0; a < NACC; ++a) {
+      const int o = tid + a * NT;
+      if (o < nout) {
+        const int r0 = (o / vq) << 2;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float inv = 1.0f / l_s[r0 + k];
+          acc[a][k].x *= inv; acc[a][k].y *= inv; acc[a][k].z *= inv; acc[a][k].w *= inv;
+        }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int a = 0; a < NACC; ++a) {
+      const int o = tid + a * NT;
+      if (o < nout) {
+        const int rb = o / vq, c4 = o - rb * vq;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) *reinterpret_cast<float4*>(sm + ((rb << 2) + k) * V4 + 4 * c4) = acc[a][k];   // [R][V4]
+      }
+    }
+    __syncthreads();
+    const int HM = H / maps;   // heads of this CTA
+    for (int u = warp; u < n * HM; u += NT / 32) {
+      const int i = u / HM, h = u - i * HM;
+      const float* a1 = sm + (2 * h * BQ + i) * V4;
+      combine_maps(p, a1, a1 + BQ * V4, row0 + i, h0 / maps + h);
+    }
+    return;
+  }
 #pragma unroll
   for (int a = 0; a < NACC; ++a) {
     const int o = tid + a * NT;
@@ -699,11 +789,56 @@ __global__ void __launch_bounds__(128) paged_attn_merge_kernel(const vila_paged_
   }
 }
 
+// one CTA per (decoded row, head) of differential attention: both maps' partial triples in split order, then the pair
+__global__ void __launch_bounds__(128) paged_attn_merge_maps_kernel(const vila_paged_attn_params p) {
+  extern __shared__ float o_s[];   // [V] a1 - lambda a2 | [4] partial sums of squares
+  const int* tile = p.tiles + 4 * blockIdx.x;
+  const int row = tile[0], h = blockIdx.y, V = p.vdim, ns = p.nsplit, HT = 2 * p.H;
+  const float* part = p.partial + (static_cast<size_t>(row) * ns * HT + 2 * h) * (V + 2);
+  const size_t stride = static_cast<size_t>(HT) * (V + 2);
+  float mx[2], inv[2];
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const float* pm = part + m * (V + 2) + V;
+    mx[m] = kNegBig;
+    for (int s = 0; s < ns; ++s) mx[m] = fmaxf(mx[m], pm[s * stride]);
+    float den = 0.f;
+    for (int s = 0; s < ns; ++s) den += expf(pm[s * stride] - mx[m]) * pm[s * stride + 1];
+    inv[m] = 1.0f / den;
+  }
+  float ss = 0.f;
+  for (int k = threadIdx.x; k < V; k += blockDim.x) {
+    float a[2] = {0.f, 0.f};
+    for (int s = 0; s < ns; ++s)
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        const float* pm = part + s * stride + m * (V + 2);
+        a[m] += expf(pm[V] - mx[m]) * pm[k];
+      }
+    const float o = fmaf(-p.diff_lambda, a[1] * inv[1], a[0] * inv[0]);
+    o_s[k] = o;
+    ss = fmaf(o, o, ss);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) o_s[V + (threadIdx.x >> 5)] = ss;
+  __syncthreads();
+  ss = (o_s[V] + o_s[V + 1]) + (o_s[V + 2] + o_s[V + 3]);
+  const float r = p.diff_scale / sqrtf(ss / static_cast<float>(V) + p.diff_eps) * out_gate(p, row, h);
+  for (int k = threadIdx.x; k < V; k += blockDim.x)
+    st_any(p.out, p.out_dtype, (static_cast<size_t>(row) * p.H + h) * V + k, o_s[k] * r);
+}
+
+// H, G: heads of the CTA (of the model, maps not counted singly)
 size_t attn_smem(const vila_paged_attn_params& p, int BQ, int BK, int H = 0, int G = 0) {
   if (H == 0) { H = p.H; G = p.G; }
+  const int maps = maps_of(p.maps), GV = G;
+  H *= maps;
+  G *= maps;
   const int D4 = round4(p.dim), V4 = round4(p.vdim), R = BQ * H;
-  return sizeof(float) * (static_cast<size_t>(R) * D4 + static_cast<size_t>(BK) * key_stride(G, D4 + 4) +
-                          static_cast<size_t>(BK) * G * V4 + 2 * static_cast<size_t>(R) * BK + H * H + 3 * R);
+  const size_t work = static_cast<size_t>(R) * D4 + static_cast<size_t>(BK) * key_stride(G, D4 + 4) +
+                      static_cast<size_t>(BK) * GV * V4 + 2 * static_cast<size_t>(R) * BK + H * H + 3 * R;
+  const size_t rows = maps > 1 ? static_cast<size_t>(R) * V4 : 0;   // the maps' finished rows, over the same memory
+  return sizeof(float) * (work > rows ? work : rows);
 }
 
 }  // namespace
@@ -712,7 +847,7 @@ int rope_append(const vila_rope_append_params& p, cudaStream_t stream) {
   if (p.T <= 0) return 0;
   VB_CHECK(p.H >= 1 && p.G >= 1 && p.dim >= 1 && p.vdim >= 1 && p.rot_dims >= 0 && p.rot_dims <= p.dim &&
                p.rot_dims % 2 == 0 && (p.rot_dims == 0 || p.inv_freq != nullptr) && (!p.v_from_k || p.vdim == p.dim) &&
-               (p.rot_layout == 0 || p.rot_layout == 1),
+               (p.rot_layout == 0 || p.rot_layout == 1) && p.maps >= 0 && p.maps <= 2 && (p.maps < 2 || !p.v_from_k),
            "rope_append: H=%d G=%d dim=%d vdim=%d rot_dims=%d v_from_k=%d", p.H, p.G, p.dim, p.vdim, p.rot_dims,
            p.v_from_k);
   VB_CUDA(launch_serial(rope_append_kernel, dim3(p.T), dim3(kThreads), sizeof(float) * (p.rot_dims + 2), stream, p));
@@ -730,22 +865,25 @@ int paged_attention(const vila_paged_attn_params& p, cudaStream_t stream) {
   VB_CHECK(p.softcap >= 0.f, "paged_attention: softcap=%f", p.softcap);
   VB_CHECK(p.window >= 0 && p.keep_first >= 0 && (p.talk_after == 0 || (p.talk != nullptr && p.sink == nullptr)),
            "paged_attention: window=%d keep_first=%d; talk_after needs talk and no sink", p.window, p.keep_first);
+  VB_CHECK(p.maps >= 0 && p.maps <= 2 &&
+               (p.maps < 2 || (p.talk == nullptr && p.sink == nullptr && p.dist_bias == nullptr && p.head_scale == nullptr)),
+           "paged_attention: maps=%d (two maps per head take no head mixing, sink, distance bias or head scale)", p.maps);
   VB_CHECK(p.max_rows >= 1 && p.max_rows <= 16 && (p.nsplit == 1 || p.max_rows == 1),
            "paged_attention: max_rows=%d nsplit=%d (key splitting serves one-row tiles)", p.max_rows, p.nsplit);
   AttnShape sh;
   sh.phase = -1;
   // Without head mixing the K/V-head groups are independent: a CTA then serves ONE K/V head and its query heads, holds
   // a quarter .. an eighth of the K | V block, and takes more rows of the sequence instead.
-  sh.hsplit = (p.talk == nullptr && p.max_rows > 1) ? p.G : 1;
-  const int Hl = p.H / sh.hsplit, Gl = p.G / sh.hsplit;
-  if (p.max_rows > 1 && Hl <= 32) {
+  sh.hsplit = p.talk == nullptr ? p.G : 1;
+  const int maps = maps_of(p.maps), Hl = p.H / sh.hsplit, Gl = p.G / sh.hsplit, Sl = Hl * maps;   // Sl: score heads of a CTA
+  if (p.max_rows > 1 && Sl <= 32) {
     // prompt portions: the register-tiled kernel, 4 .. 16 rows per CTA (about 64 score rows, 128 at most)
     sh.BQ = 16;
-    while (sh.BQ > 4 && sh.BQ * Hl > 64) sh.BQ >>= 1;
+    while (sh.BQ > 4 && sh.BQ * Sl > 64) sh.BQ >>= 1;
     sh.BK = 32;
     while (attn_smem(p, sh.BQ, sh.BK, Hl, Gl) > kSmemMax && sh.BK > 8) sh.BK >>= 1;
     const size_t smem4 = attn_smem(p, sh.BQ, sh.BK, Hl, Gl);
-    const int items = (sh.BQ * Hl / 4) * (round4(p.vdim) >> 2);      // accumulator items (4 rows x 4 columns)
+    const int items = (sh.BQ * Sl / 4) * (round4(p.vdim) >> 2);      // accumulator items (4 rows x 4 columns)
     // 512 threads (16 warps on the SM, 2-row score tiles) when there is accumulator work for them
     const int nt = items >= 512 ? 512 : 256;
     const int nacc4 = (items + nt - 1) / nt;
@@ -770,20 +908,19 @@ int paged_attention(const vila_paged_attn_params& p, cudaStream_t stream) {
     }
   }
   // decoded tokens (one-row tiles, keys optionally split over CTAs) and shapes the tiled kernel does not take
-  sh.hsplit = 1;
   sh.BQ = 1;
   while (sh.BQ < p.max_rows) sh.BQ <<= 1;
-  while (sh.BQ > 1 && sh.BQ * p.H > 64) sh.BQ >>= 1;
+  while (sh.BQ > 1 && sh.BQ * Sl > 64) sh.BQ >>= 1;
   sh.BK = 32;
-  while (attn_smem(p, sh.BQ, sh.BK) > kSmemMax && sh.BK > 4) sh.BK >>= 1;
-  while (attn_smem(p, sh.BQ, sh.BK) > kSmemMax && sh.BQ > 1) sh.BQ >>= 1;
-  const size_t smem = attn_smem(p, sh.BQ, sh.BK);
+  while (attn_smem(p, sh.BQ, sh.BK, Hl, Gl) > kSmemMax && sh.BK > 4) sh.BK >>= 1;
+  while (attn_smem(p, sh.BQ, sh.BK, Hl, Gl) > kSmemMax && sh.BQ > 1) sh.BQ >>= 1;
+  const size_t smem = attn_smem(p, sh.BQ, sh.BK, Hl, Gl);
   VB_CHECK(smem <= kSmemMax, "paged_attention: H=%d G=%d dim=%d vdim=%d need %zu bytes of shared memory", p.H, p.G,
            p.dim, p.vdim, smem);
   sh.sub = (p.max_rows + sh.BQ - 1) / sh.BQ;
-  const int nacc = (sh.BQ * p.H * (round4(p.vdim) >> 2) + kThreads - 1) / kThreads;
+  const int nacc = (sh.BQ * Sl * (round4(p.vdim) >> 2) + kThreads - 1) / kThreads;
   VB_CHECK(nacc <= 16, "paged_attention: H=%d vdim=%d: %d accumulators per thread", p.H, p.vdim, nacc);
-  const dim3 grid(p.ntiles, sh.sub, p.nsplit);
+  const dim3 grid(p.ntiles, sh.sub * sh.hsplit, p.nsplit);
 #define VB_PAGED(N)                                                                                              \
   do {                                                                                                           \
     if (smem > 48 * 1024)                                                                                        \
@@ -802,7 +939,9 @@ int paged_attention(const vila_paged_attn_params& p, cudaStream_t stream) {
     else VB_PAGED(16);
   }
 #undef VB_PAGED
-  if (p.nsplit > 1)
+  if (p.nsplit > 1 && maps > 1)
+    VB_CUDA(launch_serial(paged_attn_merge_maps_kernel, dim3(p.ntiles, p.H), dim3(128), sizeof(float) * (p.vdim + 4), stream, p));
+  else if (p.nsplit > 1)
     VB_CUDA(launch_serial(paged_attn_merge_kernel, dim3(p.ntiles, p.H), dim3(128), 0, stream, p));
   return 0;
 }

@@ -285,11 +285,11 @@ gelu_mul_gather_kernel(const void* __restrict__ z, int z_dt, const void* __restr
   }
 }
 
-// ---- sigmoid router with group-limited choice -------------------------------------------------------
-// Logits as in moe_route_kernel (fp32 dot products over the row).  Then one warp per token: scores
-// s = sigmoid(z); choice c = s + correction; group score = sum of the two largest c of the group; the
+// ---- sigmoid / softmax router with group-limited choice ----------------------------------------------
+// Logits in fp32 dot products over the row.  Then one warp per token: scores s = sigmoid(z) or softmax(z);
+// choice c = s + correction; group score = the largest c of the group or the sum of its two largest; the
 // `keep` best groups stay, the others' c become -inf; `top` rounds of arg-max over c (ties: lower index);
-// the weight of a chosen expert is its s.
+// the weight of a chosen expert is scale * s.
 __device__ __forceinline__ void warp_argmax(float& best, int& bi) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -299,29 +299,75 @@ __device__ __forceinline__ void warp_argmax(float& best, int& bi) {
   }
 }
 
-template <int TPR>
-__global__ void __launch_bounds__(kRowThreads)
-moe_route_sigmoid_kernel(const void* __restrict__ x, int x_dt, int64_t ldx, const float* __restrict__ wr,
-                         const float* __restrict__ corr, int32_t* __restrict__ idx, float* __restrict__ weight,
-                         int rows, int cols, int experts, int top, int groups, int keep) {
+// four consecutive elements (16-byte aligned fp32, 8-byte aligned bf16)
+__device__ __forceinline__ float4 ld4_any(const void* p, int dt, size_t i) {
+  if (dt) return *reinterpret_cast<const float4*>(static_cast<const float*>(p) + i);
+  const uint2 u = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p) + i);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                     __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void st4_any(void* p, int dt, size_t i, float4 v) {
+  if (dt) {
+    *reinterpret_cast<float4*>(static_cast<float*>(p) + i) = v;
+    return;
+  }
+  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<unsigned int*>(&lo);
+  u.y = *reinterpret_cast<unsigned int*>(&hi);
+  *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p) + i) = u;
+}
+
+// A warp takes four outputs at a time (their dot products share the row's loads and overlap); the shared expert's gate,
+// if there is one, is the output after the last.
+template <int TPR, bool VEC>
+__global__ void __launch_bounds__(kRowThreads) moe_route_scores_kernel(const vila_moe_route_params p) {
   extern __shared__ float z_s[];  // per token: s [experts] | c [experts] | group score [groups]
   const int wid = threadIdx.x >> 5, lane = lane_id();
   const int row = row_of<TPR>();
-  if (row >= rows) return;
-  const int per_tok = 2 * experts + groups;
-  float* s = TPR == 32 ? z_s + wid * per_tok : z_s;
+  if (row >= p.rows) return;
+  const int experts = p.experts, groups = p.groups, keep = p.keep, cols = p.cols;
+  float* s = TPR == 32 ? z_s + wid * (2 * experts + groups) : z_s;
   float* c = s + experts;
   float* gs = c + experts;
-  const size_t xb = static_cast<size_t>(row) * ldx;
-  for (int e = (TPR == 32 ? 0 : wid); e < experts; e += (TPR == 32 ? 1 : kRowsPerCta)) {
-    const float* we = wr + static_cast<size_t>(e) * cols;
-    float a = 0.f;
-    for (int k = lane; k < cols; k += 32) a += ld_any(x, x_dt, xb + k) * we[k];
-    a = warp_sum(a);
+  const size_t xb = static_cast<size_t>(row) * p.ldx;
+  const int outs = experts + (p.gate_w ? 1 : 0);
+  for (int e0 = 4 * (TPR == 32 ? 0 : wid); e0 < outs; e0 += 4 * (TPR == 32 ? 1 : kRowsPerCta)) {
+    const float* we[4];
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int e = min(e0 + u, outs - 1);
+      we[u] = e < experts ? p.w + static_cast<size_t>(e) * cols : p.gate_w;
+    }
+    if (VEC) {
+      for (int k = 4 * lane; k < cols; k += 128) {
+        const float4 xv = ld4_any(p.x, p.x_dtype, xb + k);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const float4 wv = __ldg(reinterpret_cast<const float4*>(we[u] + k));
+          a[u] = fmaf(xv.x, wv.x, a[u]); a[u] = fmaf(xv.y, wv.y, a[u]);
+          a[u] = fmaf(xv.z, wv.z, a[u]); a[u] = fmaf(xv.w, wv.w, a[u]);
+        }
+      }
+    } else {
+      for (int k = lane; k < cols; k += 32) {
+        const float xv = ld_any(p.x, p.x_dtype, xb + k);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) a[u] = fmaf(xv, we[u][k], a[u]);
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) a[u] += __shfl_xor_sync(0xffffffffu, a[u], o);
     if (lane == 0) {
-      const float sv = sigmoid_f(a);
-      s[e] = sv;
-      c[e] = sv + (corr ? corr[e] : 0.f);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int e = e0 + u;
+        if (e < experts) s[e] = a[u];
+        else if (e < outs) p.gate[row] = sigmoid_f(a[u]);
+      }
     }
   }
   if (TPR == 32) __syncwarp();
@@ -329,6 +375,21 @@ moe_route_sigmoid_kernel(const void* __restrict__ x, int x_dt, int64_t ldx, cons
     __syncthreads();
     if (wid != 0) return;
   }
+  float mx = 0.f, inv = 1.f;
+  if (p.score == VILA_SCORE_SOFTMAX) {
+    mx = -INFINITY;
+    for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, s[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < experts; e += 32) sum += expf(s[e] - mx);
+    inv = 1.0f / warp_sum(sum);
+  }
+  for (int e = lane; e < experts; e += 32) {   // a lane rewrites the entries that it read
+    const float sv = p.score == VILA_SCORE_SOFTMAX ? expf(s[e] - mx) * inv : sigmoid_f(s[e]);
+    s[e] = sv;
+    c[e] = sv + (p.correction ? p.correction[e] : 0.f);
+  }
+  __syncwarp();
   const int gsize = experts / groups;
   if (keep < groups) {
     for (int g = lane; g < groups; g += 32) {
@@ -338,7 +399,7 @@ moe_route_sigmoid_kernel(const void* __restrict__ x, int x_dt, int64_t ldx, cons
         if (v > a) { b = a; a = v; }
         else if (v > b) b = v;
       }
-      gs[g] = gsize >= 2 ? a + b : a;
+      gs[g] = (p.group_top >= 2 && gsize >= 2) ? a + b : a;
     }
     __syncwarp();
     // `keep` rounds of arg-max over the groups; a kept group is marked by +inf
@@ -357,7 +418,7 @@ moe_route_sigmoid_kernel(const void* __restrict__ x, int x_dt, int64_t ldx, cons
       if (gs[e / gsize] != INFINITY) c[e] = -INFINITY;
     __syncwarp();
   }
-  for (int j = 0; j < top; ++j) {
+  for (int j = 0; j < p.top; ++j) {
     float best = -INFINITY;
     int bi = 0x7fffffff;
     for (int e = lane; e < experts; e += 32) {
@@ -367,8 +428,8 @@ moe_route_sigmoid_kernel(const void* __restrict__ x, int x_dt, int64_t ldx, cons
     warp_argmax(best, bi);
     if (bi == 0x7fffffff) bi = 0;   // fewer selectable experts than `top` (refused by the launcher's callers)
     if (lane == 0) {
-      idx[static_cast<size_t>(row) * top + j] = bi;
-      weight[static_cast<size_t>(row) * top + j] = s[bi];
+      p.idx[static_cast<size_t>(row) * p.top + j] = bi;
+      p.weight[static_cast<size_t>(row) * p.top + j] = p.scale * s[bi];
       c[bi] = -INFINITY;
     }
     __syncwarp();
@@ -455,24 +516,6 @@ struct ScaledResidual {
   float eps;
 };
 
-__device__ __forceinline__ float4 ld4_any(const void* p, int dt, size_t i) {
-  if (dt) return *reinterpret_cast<const float4*>(static_cast<const float*>(p) + i);
-  const uint2 u = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p) + i);
-  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
-                     __uint_as_float(u.y & 0xffff0000u));
-}
-__device__ __forceinline__ void st4_any(void* p, int dt, size_t i, float4 v) {
-  if (dt) {
-    *reinterpret_cast<float4*>(static_cast<float*>(p) + i) = v;
-    return;
-  }
-  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-  uint2 u;
-  u.x = *reinterpret_cast<unsigned int*>(&lo);
-  u.y = *reinterpret_cast<unsigned int*>(&hi);
-  *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p) + i) = u;
-}
-
 template <int TPR>
 __global__ void __launch_bounds__(kRowThreads) scaled_residual_norm_kernel(const ScaledResidual p) {
   __shared__ float red[kRowsPerCta];
@@ -537,37 +580,120 @@ __global__ void __launch_bounds__(kRowThreads) scaled_residual_norm_vec_kernel(c
   }
 }
 
-// ---- read-out of a recurrent mixer: per-head RMS norm, shared weight, SiLU gate ---------------------------
-// out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * w * silu(gate[t, h, :]); a warp per (token, head)
-template <bool VEC>
+// ---- read-out of a recurrent mixer: per-head RMS norm, shared weight, gate -----------------------------------
+// out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * w * act(gate[t, h, :]), act = SiLU or sigmoid; a warp per
+// (token, head), or a CTA where a head is wide
+template <int TPR, bool VEC>
 __global__ void __launch_bounds__(kRowThreads)
 gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, const void* __restrict__ gate, int g_dt,
-                       int64_t ldg, float eps, void* __restrict__ out, int o_dt, int pairs, int H, int vdim) {
-  const int pair = blockIdx.x * kRowsPerCta + (threadIdx.x >> 5);
+                       int64_t ldg, float eps, void* __restrict__ out, int o_dt, int pairs, int H, int vdim, int gate_act) {
+  __shared__ float red[kRowsPerCta];
+  const int pair = row_of<TPR>();
   if (pair >= pairs) return;
-  const int t = pair / H, h = pair - t * H, lane = threadIdx.x & 31;
+  const int t = pair / H, h = pair - t * H, l = col0_of<TPR>();
   const size_t ob = static_cast<size_t>(pair) * vdim, gb = static_cast<size_t>(t) * ldg + static_cast<size_t>(h) * vdim;
+  auto act = [&](float z) { return gate_act == VILA_ACT_SIGMOID ? sigmoid_f(z) : silu_exact_f(z); };
   float ss = 0.f;
   if (VEC) {
-    for (int c = 4 * lane; c < vdim; c += 128) {
+    for (int c = 4 * l; c < vdim; c += 4 * TPR) {
       const float4 v = *reinterpret_cast<const float4*>(o + ob + c);
       ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
     }
   } else {
-    for (int c = lane; c < vdim; c += 32) ss = fmaf(o[ob + c], o[ob + c], ss);
+    for (int c = l; c < vdim; c += TPR) ss = fmaf(o[ob + c], o[ob + c], ss);
   }
-  ss = warp_sum(ss);
+  ss = row_sum<TPR>(ss, red);
   const float r = 1.0f / sqrtf(ss / static_cast<float>(vdim) + eps);
   if (VEC) {
-    for (int c = 4 * lane; c < vdim; c += 128) {
+    for (int c = 4 * l; c < vdim; c += 4 * TPR) {
       const float4 v = *reinterpret_cast<const float4*>(o + ob + c), g = ld4_any(gate, g_dt, gb + c);
       const float4 w4 = __ldg(reinterpret_cast<const float4*>(w + c));
-      st4_any(out, o_dt, ob + c, make_float4(v.x * r * w4.x * silu_exact_f(g.x), v.y * r * w4.y * silu_exact_f(g.y),
-                                             v.z * r * w4.z * silu_exact_f(g.z), v.w * r * w4.w * silu_exact_f(g.w)));
+      st4_any(out, o_dt, ob + c, make_float4(v.x * r * w4.x * act(g.x), v.y * r * w4.y * act(g.y),
+                                             v.z * r * w4.z * act(g.z), v.w * r * w4.w * act(g.w)));
     }
   } else {
-    for (int c = lane; c < vdim; c += 32)
-      st_any(out, o_dt, ob + c, o[ob + c] * r * w[c] * silu_exact_f(ld_any(gate, g_dt, gb + c)));
+    for (int c = l; c < vdim; c += TPR)
+      st_any(out, o_dt, ob + c, o[ob + c] * r * w[c] * act(ld_any(gate, g_dt, gb + c)));
+  }
+}
+
+// ---- parallel-sublayer residual + Dynamic Tanh norms (elementwise: nothing is reduced over the row) -----------
+// x (or an embedding row) += mult * (sa * a + sb * (b * gate + routed partials, identity experts included)), then up to two
+// norms tanh(alpha x) * w + bias of the result; V = 4 or 1 neighbouring columns per thread
+template <int V>
+struct Cols {
+  float v[V];
+};
+template <int V>
+__device__ __forceinline__ Cols<V> ldv(const void* p, int dt, size_t i) {
+  Cols<V> r;
+  if (V == 4) {
+    const float4 u = ld4_any(p, dt, i);
+    r.v[0] = u.x; r.v[V == 4 ? 1 : 0] = u.y; r.v[V == 4 ? 2 : 0] = u.z; r.v[V == 4 ? 3 : 0] = u.w;
+  } else {
+    r.v[0] = ld_any(p, dt, i);
+  }
+  return r;
+}
+template <int V>
+__device__ __forceinline__ void stv(void* p, int dt, size_t i, const Cols<V>& c) {
+  if (V == 4) st4_any(p, dt, i, make_float4(c.v[0], c.v[V == 4 ? 1 : 0], c.v[V == 4 ? 2 : 0], c.v[V == 4 ? 3 : 0]));
+  else st_any(p, dt, i, c.v[0]);
+}
+
+template <int V>
+__global__ void __launch_bounds__(kRowThreads) tanh_residual_kernel(const vila_tanh_residual_params p) {
+  const int cv = p.cols / V;
+  const size_t total = static_cast<size_t>(p.rows) * cv;
+  for (size_t i = blockIdx.x * static_cast<size_t>(kRowThreads) + threadIdx.x; i < total;
+       i += static_cast<size_t>(gridDim.x) * kRowThreads) {
+    const int r = static_cast<int>(i / cv), c = static_cast<int>(i - static_cast<size_t>(r) * cv) * V;
+    const size_t at = static_cast<size_t>(r) * p.cols + c;
+    Cols<V> x = p.table ? ldv<V>(p.table, p.table_dtype, static_cast<size_t>(p.ids[r]) * p.cols + c) : ldv<V>(p.x, VILA_DT_F32, at);
+    if (p.a) {
+      const Cols<V> a = ldv<V>(p.a, p.a_dtype, static_cast<size_t>(r) * p.lda + c), sa = ldv<V>(p.a_scale, VILA_DT_F32, c);
+      Cols<V> y;
+#pragma unroll
+      for (int k = 0; k < V; ++k) y.v[k] = sa.v[k] * a.v[k];
+      if (p.b || p.part) {
+        Cols<V> f;
+#pragma unroll
+        for (int k = 0; k < V; ++k) f.v[k] = 0.f;
+        if (p.b) {
+          const float g = p.b_gate ? p.b_gate[r] : 1.0f;
+          const Cols<V> b = ldv<V>(p.b, p.b_dtype, static_cast<size_t>(r) * p.ldb + c);
+#pragma unroll
+          for (int k = 0; k < V; ++k) f.v[k] = g * b.v[k];
+        }
+        if (p.part) {
+          const size_t pr = static_cast<size_t>(r) * p.n_partials;
+          for (int j = 0; j < p.n_partials; ++j) {
+            const bool self = p.idx != nullptr && p.idx[pr + j] >= p.experts;
+            const float w = self ? p.weight[pr + j] : 1.0f;
+            const Cols<V> q = self ? ldv<V>(p.h, p.h_dtype, static_cast<size_t>(r) * p.ldh + c)
+                                   : ldv<V>(p.part, p.part_dtype, (pr + j) * p.ldp + c);
+#pragma unroll
+            for (int k = 0; k < V; ++k) f.v[k] = fmaf(w, q.v[k], f.v[k]);
+          }
+        }
+        const Cols<V> sb = ldv<V>(p.b_scale, VILA_DT_F32, c);
+#pragma unroll
+        for (int k = 0; k < V; ++k) y.v[k] = fmaf(sb.v[k], f.v[k], y.v[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.v[k] = fmaf(p.mult, y.v[k], x.v[k]);
+    }
+    if (p.a || p.table) stv<V>(p.x, VILA_DT_F32, at, x);
+#pragma unroll
+    for (int o = 0; o < 2; ++o) {
+      if (o < p.n_out) {
+        const Cols<V> w = ldv<V>(p.w[o], VILA_DT_F32, c), b = ldv<V>(p.bias[o], VILA_DT_F32, c);
+        Cols<V> n;
+#pragma unroll
+        for (int k = 0; k < V; ++k) n.v[k] = fmaf(tanhf(p.alpha[o] * x.v[k]), w.v[k], b.v[k]);
+        stv<V>(p.out[o], p.out_dtype, at, n);
+      }
+    }
   }
 }
 
@@ -603,18 +729,46 @@ int scaled_residual_norm_rows(float* x, const void* a, int a_dt, int64_t lda, co
 }
 
 int gated_head_norm_rows(const float* o, const float* w, const void* gate, int g_dt, int64_t ldg, float eps, void* out,
-                         int o_dt, int rows, int H, int vdim, cudaStream_t stream) {
+                         int o_dt, int rows, int H, int vdim, int gate_act, cudaStream_t stream) {
   if (rows <= 0) return 0;
   VB_CHECK(H >= 1 && vdim >= 1 && w != nullptr && gate != nullptr, "gated_head_norm_rows: H=%d vdim=%d", H, vdim);
   VB_CHECK(static_cast<long>(rows) * H < (1L << 31), "gated_head_norm_rows: rows=%d H=%d", rows, H);
+  VB_CHECK(gate_act == VILA_ACT_SILU || gate_act == VILA_ACT_SIGMOID, "gated_head_norm_rows: gate activation %d", gate_act);
   const int pairs = rows * H;
   const bool vec = vdim % 4 == 0 && aligned_to(o, 16) && aligned_to(w, 16) && rows4(gate, ldg, g_dt) && aligned_to(out, o_dt ? 16 : 8);
-  if (vec)
-    VB_CUDA(launch_serial(gated_head_norm_kernel<true>, dim3(row_grid(pairs)), dim3(kRowThreads), 0, stream, o, w, gate, g_dt,
-                          ldg, eps, out, o_dt, pairs, H, vdim));
-  else
-    VB_CUDA(launch_serial(gated_head_norm_kernel<false>, dim3(row_grid(pairs)), dim3(kRowThreads), 0, stream, o, w, gate, g_dt,
-                          ldg, eps, out, o_dt, pairs, H, vdim));
+#define VB_GHN(K, G)                                                                                                      \
+  VB_CUDA(launch_serial(K, dim3(G), dim3(kRowThreads), 0, stream, o, w, gate, g_dt, ldg, eps, out, o_dt, pairs, H, vdim, gate_act))
+  if (vdim >= kWideCols) {
+    if (vec) VB_GHN((gated_head_norm_kernel<256, true>), pairs);
+    else VB_GHN((gated_head_norm_kernel<256, false>), pairs);
+  } else if (vec) {
+    VB_GHN((gated_head_norm_kernel<32, true>), row_grid(pairs));
+  } else {
+    VB_GHN((gated_head_norm_kernel<32, false>), row_grid(pairs));
+  }
+#undef VB_GHN
+  return 0;
+}
+
+int tanh_residual_rows(const vila_tanh_residual_params& p, cudaStream_t stream) {
+  if (p.rows <= 0) return 0;
+  VB_CHECK(p.cols > 0 && p.x != nullptr && p.n_out >= 0 && p.n_out <= 2 && (p.table == nullptr || p.ids != nullptr),
+           "tanh_residual_rows: cols=%d n_out=%d", p.cols, p.n_out);
+  VB_CHECK((p.a == nullptr || p.a_scale != nullptr) && ((p.b == nullptr && p.part == nullptr) || (p.a != nullptr && p.b_scale != nullptr)),
+           "tanh_residual_rows: a branch without its scale, or a second branch without the first");
+  VB_CHECK(p.part == nullptr || (p.n_partials >= 1 && (p.idx == nullptr || (p.weight != nullptr && p.h != nullptr))),
+           "tanh_residual_rows: n_partials=%d; indices need weights and the experts' input", p.n_partials);
+  bool vec = p.cols % 4 == 0 && aligned_to(p.x, 16) && (!p.table || aligned_to(p.table, p.table_dtype ? 16 : 8)) &&
+             (!p.a || (rows4(p.a, p.lda, p.a_dtype) && aligned_to(p.a_scale, 16))) && (!p.b || rows4(p.b, p.ldb, p.b_dtype)) &&
+             (!p.part || rows4(p.part, p.ldp, p.part_dtype)) && (!p.h || rows4(p.h, p.ldh, p.h_dtype)) &&
+             (!p.b_scale || aligned_to(p.b_scale, 16));
+  for (int k = 0; k < p.n_out; ++k) {
+    VB_CHECK(p.w[k] != nullptr && p.bias[k] != nullptr && p.out[k] != nullptr, "tanh_residual_rows: norm %d is incomplete", k);
+    vec = vec && aligned_to(p.w[k], 16) && aligned_to(p.bias[k], 16) && aligned_to(p.out[k], p.out_dtype ? 16 : 8);
+  }
+  const size_t total = static_cast<size_t>(p.rows) * (vec ? p.cols / 4 : p.cols);
+  if (vec) VB_CUDA(launch_serial(tanh_residual_kernel<4>, dim3(flat_grid(total)), dim3(kRowThreads), 0, stream, p));
+  else VB_CUDA(launch_serial(tanh_residual_kernel<1>, dim3(flat_grid(total)), dim3(kRowThreads), 0, stream, p));
   return 0;
 }
 
@@ -719,21 +873,25 @@ int gelu_mul_gather(const void* z, int z_dt, const void* table, int dt, int64_t 
   return 0;
 }
 
-int moe_route_sigmoid(const void* x, int x_dt, int64_t ldx, const float* wr, const float* corr, int32_t* idx,
-                      float* weight, int rows, int cols, int experts, int top, int groups, int keep,
-                      cudaStream_t stream) {
-  if (rows <= 0) return 0;
-  VB_CHECK(experts >= 1 && experts <= 1024 && groups >= 1 && experts % groups == 0 && keep >= 1 && keep <= groups &&
-               top >= 1 && top <= keep * (experts / groups),
-           "moe_route_sigmoid: experts=%d top=%d groups=%d keep=%d", experts, top, groups, keep);
-  const size_t per_tok = sizeof(float) * (2 * experts + groups);
-  if (rows <= 1024 || per_tok * kRowsPerCta > 48 * 1024)   // few tokens, or too many experts for a warp's share
-    VB_CUDA(launch_serial(moe_route_sigmoid_kernel<256>, dim3(rows), dim3(kRowThreads), per_tok, stream, x, x_dt,
-                          ldx, wr, corr, idx, weight, rows, cols, experts, top, groups, keep));
-  else
-    VB_CUDA(launch_serial(moe_route_sigmoid_kernel<32>, dim3(row_grid(rows)), dim3(kRowThreads),
-                          per_tok * kRowsPerCta, stream, x, x_dt, ldx, wr, corr, idx, weight, rows, cols, experts,
-                          top, groups, keep));
+int moe_route_scores(const vila_moe_route_params& p, cudaStream_t stream) {
+  if (p.rows <= 0) return 0;
+  VB_CHECK(p.experts >= 1 && p.experts <= 1024 && p.groups >= 1 && p.experts % p.groups == 0 && p.keep >= 1 &&
+               p.keep <= p.groups && p.top >= 1 && p.top <= p.keep * (p.experts / p.groups),
+           "moe_route_scores: experts=%d top=%d groups=%d keep=%d", p.experts, p.top, p.groups, p.keep);
+  VB_CHECK((p.score == VILA_SCORE_SIGMOID || p.score == VILA_SCORE_SOFTMAX) && (p.group_top == 1 || p.group_top == 2) &&
+               (p.gate_w == nullptr || p.gate != nullptr),
+           "moe_route_scores: score=%d group_top=%d", p.score, p.group_top);
+  const size_t per_tok = sizeof(float) * (2 * p.experts + p.groups);
+  const bool vec = p.cols % 4 == 0 && rows4(p.x, p.ldx, p.x_dtype) && aligned_to(p.w, 16) && (!p.gate_w || aligned_to(p.gate_w, 16));
+#define VB_ROUTE(K, G, S) VB_CUDA(launch_serial(K, dim3(G), dim3(kRowThreads), S, stream, p))
+  if (p.rows <= 1024 || per_tok * kRowsPerCta > 48 * 1024) {   // few tokens, or too many experts for a warp's share
+    if (vec) VB_ROUTE((moe_route_scores_kernel<256, true>), p.rows, per_tok);
+    else VB_ROUTE((moe_route_scores_kernel<256, false>), p.rows, per_tok);
+  } else {
+    if (vec) VB_ROUTE((moe_route_scores_kernel<32, true>), row_grid(p.rows), per_tok * kRowsPerCta);
+    else VB_ROUTE((moe_route_scores_kernel<32, false>), row_grid(p.rows), per_tok * kRowsPerCta);
+  }
+#undef VB_ROUTE
   return 0;
 }
 

@@ -8,6 +8,7 @@ from .ludazen import LudazenConfig, LudazenForCausalLM, LudazenLayerConfig
 from .lufatar import LufatarConfig, LufatarForCausalLM, LufatarLayerConfig
 from .modeling_vila import VILAForCausalLM
 from .moronex import MoronexConfig, MoronexForCausalLM, MoronexLayerConfig
+from .nibelix import NibelixConfig, NibelixForCausalLM, NibelixLayerConfig
 from .nusovik import NusovikConfig, NusovikForCausalLM, NusovikLayerConfig
 from .projector import MultimodalProjector
 from .registry import LANGUAGE_MODELS, language_model_architecture, load_language_model

@@ -12,11 +12,12 @@ from .bivizen import BivizenForCausalLM
 from .ludazen import LudazenForCausalLM
 from .lufatar import LufatarForCausalLM
 from .moronex import MoronexForCausalLM
+from .nibelix import NibelixForCausalLM
 from .nusovik import NusovikForCausalLM
 
 LANGUAGE_MODELS: Dict[str, type] = {"Moronex": MoronexForCausalLM, "Lufatar": LufatarForCausalLM,
                                     "Nusovik": NusovikForCausalLM, "Ludazen": LudazenForCausalLM,
-                                    "Bivizen": BivizenForCausalLM}
+                                    "Bivizen": BivizenForCausalLM, "Nibelix": NibelixForCausalLM}
 
 _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.float32, "fp32": torch.float32}
 

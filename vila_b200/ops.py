@@ -14,6 +14,7 @@ from . import _lib
 from ._lib import DecodeAttnParams, DecodeAttnSplitParams, FmhaParams, GemvParams, check
 
 ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF, ACT_SILU = 0, 1, 2, 3
+FLAG_GEGLU = 8
 
 
 def _stream() -> int:
@@ -50,17 +51,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
            swiglu: bool = False, out: Optional[torch.Tensor] = None,
            block_n: Optional[int] = None, static_w: bool = False,
            act_params: Optional[Tuple[float, float]] = None,
-           glu_clamp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+           glu_clamp: Optional[Tuple[float, float]] = None, geglu: bool = False) -> torch.Tensor:
     """out = epilogue(x @ w.T).  x [M,K] (row stride arbitrary), w [N,K].
     static_w: w is a parameter (VILA_FLAG_STATIC_W): it may be fetched before the PDL wait.
     act_params: the two coefficients of ACT_XIELU (positive side, negative side).
-    glu_clamp = (alpha, limit): clamped gated unit over interleaved (gate, up) weight rows, see VILA_FLAG_GLU_CLAMP."""
+    glu_clamp = (alpha, limit): clamped gated unit over interleaved (gate, up) weight rows, see VILA_FLAG_GLU_CLAMP.
+    geglu: gelu_tanh(gate) * up over interleaved rows."""
     _chk(x, "x"); _chk(w, "w")
     assert x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1], (x.shape, w.shape)
     assert x.stride(1) == 1 and w.stride(1) == 1
     M, K = x.shape
     N = w.shape[0]
-    n_out = N // 2 if (swiglu or glu_clamp is not None) else N
+    n_out = N // 2 if (swiglu or geglu or glu_clamp is not None) else N
     if out is None:
         out = torch.empty((M, n_out), dtype=torch.bfloat16, device=x.device)
     else:
@@ -75,7 +77,11 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     lib = _lib.load()
     args = (_p(x), x.stride(0), _p(w), w.stride(0), _p(bias), _p(residual), ld_res, res_row_mod,
             _p(out), out.stride(0), M, N, K, act, (1 if swiglu else 0) | (2 if static_w else 0), _stream())
-    if glu_clamp is not None:
+    if geglu:
+        assert residual is None and block_n is None and act == ACT_NONE and not swiglu and glu_clamp is None
+        check(lib.vila_linear_act(_p(x), x.stride(0), _p(w), w.stride(0), _p(bias), _p(out), out.stride(0), M, N, K,
+                                  act, 0.0, 0.0, FLAG_GEGLU | (2 if static_w else 0), _stream()), "vila_linear_act")
+    elif glu_clamp is not None:
         assert residual is None and block_n is None and act == ACT_NONE and not swiglu
         check(lib.vila_linear_act(_p(x), x.stride(0), _p(w), w.stride(0), _p(bias), _p(out), out.stride(0), M, N, K,
                                   act, float(glu_clamp[0]), float(glu_clamp[1]), 4 | (2 if static_w else 0), _stream()),
@@ -411,6 +417,8 @@ def decode_attention_batch(qkv: torch.Tensor, positions: torch.Tensor, k_pool: t
 DT_BF16, DT_F32 = 0, 1
 ACT_RELU2 = 4
 ACT_XIELU = 5   # z > 0: a_pos z^2 + z / 2;  z <= 0: a_neg (e^z - 1 - z) + z / 2  (act_params = (a_pos, a_neg))
+ACT_SOFTCAP = 6  # cap tanh(z / cap) (act_params = (cap, 0)); glinear only
+ACT_SIGMOID = 7  # only as a gate's activation
 _DT = {torch.bfloat16: DT_BF16, torch.float32: DT_F32}
 
 
@@ -493,19 +501,20 @@ def glinear(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = N
             seg: Optional[torch.Tensor] = None, a_rows: Optional[torch.Tensor] = None, a_row_div: int = 1,
             o_rows: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None,
             out_rows_total: Optional[int] = None, glu_clamp: Optional[Tuple[float, float]] = None,
-            act_params: Optional[Tuple[float, float]] = None, in_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+            act_params: Optional[Tuple[float, float]] = None, in_scale: Optional[torch.Tensor] = None,
+            geglu: bool = False) -> torch.Tensor:
     """Any-shape (grouped) linear layer, fp32 accumulation on the CUDA cores (vila_glinear).
     w [N, K] (groups == 1) or [groups, N, K].  Batched groups (seg None): group g reads the A columns
     [g * a_group_off, + K) and writes the output columns [g * o_group_off, + N).  Segmented (seg int32
     [groups + 1]): the rows of group g are the sorted positions seg[g]..seg[g+1]; see the header.
-    act_params: the coefficients of ACT_XIELU.  in_scale fp32: sorted position i is computed from its input row
+    act_params: the coefficients of ACT_XIELU / the cap of ACT_SOFTCAP; geglu: gelu_tanh(gate) * up over interleaved rows.  in_scale fp32: sorted position i is computed from its input row
     times in_scale[a_rows[i]] (a_rows None: in_scale[i]): the scale enters before bias and activation."""
     assert a.dim() == 2 and a.stride(1) == 1
     if w.dim() == 2:
         w = w[None]
     assert w.dim() == 3 and w.stride(2) == 1 and w.shape[0] == groups, (w.shape, groups)
     N, K = w.shape[1], w.shape[2]
-    n_out = N // 2 if (swiglu or glu_clamp is not None) else N   # glu_clamp = (alpha, limit): see VILA_FLAG_GLU_CLAMP
+    n_out = N // 2 if (swiglu or geglu or glu_clamp is not None) else N   # glu_clamp = (alpha, limit): see VILA_FLAG_GLU_CLAMP
     M = a.shape[0] if a_rows is None else a_rows.numel()
     if out is None:
         cols = n_out if seg is not None or groups == 1 else o_group_off * (groups - 1) + n_out
@@ -526,7 +535,7 @@ def glinear(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = N
         assert bias.dtype == w.dtype
     p.M, p.N, p.K, p.groups = M, N, K, groups
     p.mode = 0 if seg is None else 1
-    p.a_row_div, p.act, p.flags = a_row_div, act, (1 if swiglu else 0) | (4 if glu_clamp is not None else 0)
+    p.a_row_div, p.act, p.flags = a_row_div, act, (1 if swiglu else 0) | (4 if glu_clamp is not None else 0) | (FLAG_GEGLU if geglu else 0)
     if glu_clamp is not None or act_params is not None or in_scale is not None:
         assert in_scale is None or o_rows is None
         ext = _lib.GLinearExt(float(glu_clamp[0]) if glu_clamp else 1.0, float(glu_clamp[1]) if glu_clamp else float("inf"),
@@ -681,15 +690,16 @@ def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, tiles: tor
 def linear_any(x: torch.Tensor, w: torch.Tensor, *, swiglu: bool = False, out_dtype=None,
                bias: Optional[torch.Tensor] = None, act: int = ACT_NONE,
                act_params: Optional[Tuple[float, float]] = None,
-               glu_clamp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+               glu_clamp: Optional[Tuple[float, float]] = None, geglu: bool = False) -> torch.Tensor:
     """act(x [M, K] · w[N, K]^T + bias): bf16 operands with 16-byte aligned rows go to the tcgen05 GEMM,
     everything else (fp32 tensors, odd shapes, an fp32 result) to the CUDA-core grouped kernel."""
     N, K = w.shape
     if (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and out_dtype in (None, torch.bfloat16)
             and K % 8 == 0 and N % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
-            and (not (swiglu or glu_clamp) or N % 32 == 0)):
-        return linear(x, w, bias, act=act, swiglu=swiglu, static_w=True, act_params=act_params, glu_clamp=glu_clamp)
-    return glinear(x, w, swiglu=swiglu, out_dtype=out_dtype, bias=bias, act=act, act_params=act_params, glu_clamp=glu_clamp)
+            and (not (swiglu or glu_clamp or geglu) or N % 32 == 0)):
+        return linear(x, w, bias, act=act, swiglu=swiglu, static_w=True, act_params=act_params, glu_clamp=glu_clamp, geglu=geglu)
+    return glinear(x, w, swiglu=swiglu, out_dtype=out_dtype, bias=bias, act=act, act_params=act_params, glu_clamp=glu_clamp,
+                   geglu=geglu)
 
 
 def embed_pair_rows(table: torch.Tensor, pair_table: torch.Tensor, ids: torch.Tensor, prev_ids: torch.Tensor,
@@ -768,20 +778,22 @@ def rope_append(qkv: torch.Tensor, positions: torch.Tensor, cache_rows: torch.Te
                 heads: int, kv_heads: int, dim: int, vdim: int, inv_freq: Optional[torch.Tensor],
                 unit_norm: bool, eps: float, q_norm_w: Optional[torch.Tensor] = None,
                 k_norm_w: Optional[torch.Tensor] = None, v_from_k: bool = False, halves: bool = False,
-                mscale: float = 1.0, v_first: Optional[torch.Tensor] = None, v_mix: float = 0.0) -> torch.Tensor:
+                mscale: float = 1.0, v_first: Optional[torch.Tensor] = None, v_mix: float = 0.0,
+                maps: int = 1) -> torch.Tensor:
     """qkv [T, >= heads*dim + kv_heads*(dim+vdim)] -> q fp32 [T, heads*dim] (rotated, unit-normed); the
     token's k | v go to row cache_rows[t] of pool [pool rows, kv_heads*(dim+vdim)].  inv_freq float64
     [rot_dims / 2] (None: no rotation).  q_norm_w / k_norm_w fp32 [dim]: weights of the per-head norm.
     v_from_k: qkv holds q | k only, the cached value of a token is its incoming key (before rotation / norm).
     halves: column i of the rotated part pairs with i + rot_dims / 2 instead of 2i with 2i + 1; mscale multiplies
     cos and sin (a magnitude correction of rescaled frequencies).  v_first [T, kv_heads*vdim] (a view with a row
-    stride is fine): the cached value is (1 - v_mix) v + v_mix v_first."""
-    assert qkv.dim() == 2 and qkv.stride(1) == 1
-    assert qkv.shape[1] >= heads * dim + kv_heads * (dim if v_from_k else dim + vdim)
+    stride is fine): the cached value is (1 - v_mix) v + v_mix v_first.  maps = 2: q and k heads are two maps of dim columns
+    each (differential attention): q [T, heads*2*dim], pool rows k (kv_heads*2*dim) | v."""
+    assert qkv.dim() == 2 and qkv.stride(1) == 1 and (maps == 1 or not v_from_k)
+    assert qkv.shape[1] >= heads * maps * dim + kv_heads * (dim if v_from_k else maps * dim + vdim)
     assert not v_from_k or vdim == dim
-    assert pool.dim() == 2 and pool.is_contiguous() and pool.shape[1] == kv_heads * (dim + vdim)
+    assert pool.dim() == 2 and pool.is_contiguous() and pool.shape[1] == kv_heads * (maps * dim + vdim)
     T = qkv.shape[0]
-    q = torch.empty(T, heads * dim, dtype=torch.float32, device=qkv.device)
+    q = torch.empty(T, heads * maps * dim, dtype=torch.float32, device=qkv.device)
     p = _lib.RopeAppendParams()
     p.qkv, p.ldq = _p(qkv), qkv.stride(0)
     p.positions, p.cache_rows = _i32(positions, "positions"), _i32(cache_rows, "cache_rows")
@@ -796,7 +808,7 @@ def rope_append(qkv: torch.Tensor, positions: torch.Tensor, cache_rows: torch.Te
     for t_ in (q_norm_w, k_norm_w):
         assert t_ is None or (unit_norm and t_.numel() == dim)
     p.q_norm_w, p.k_norm_w, p.v_from_k = _f32(q_norm_w, "q_norm_w"), _f32(k_norm_w, "k_norm_w"), 1 if v_from_k else 0
-    p.rot_layout, p.rot_mscale = 1 if halves else 0, float(mscale)
+    p.rot_layout, p.rot_mscale, p.maps = 1 if halves else 0, float(mscale), maps
     if v_first is not None:
         assert v_first.shape == (T, kv_heads * vdim) and v_first.stride(1) == 1 and not v_from_k
         p.v_first, p.ld_vf, p.v_first_dtype, p.v_mix = _p(v_first), v_first.stride(0), _dt(v_first, "v_first"), float(v_mix)
@@ -811,7 +823,7 @@ def paged_attention(q: torch.Tensor, pool: torch.Tensor, page_tables: torch.Tens
                     nsplit: int = 1, dist_bias: Optional[torch.Tensor] = None, chunk: int = 0,
                     gate: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0,
                     talk_after: bool = False, head_scale: Optional[torch.Tensor] = None,
-                    softcap: float = 0.0) -> torch.Tensor:
+                    softcap: float = 0.0, diff: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
     """Causal grouped-query attention of q fp32 [T, heads*dim] over the paged k | v pool, fp32 scores and
     softmax, optional mixing of the heads' scores (talk fp32 [heads, heads]) and per-head sink logit in
     the denominator.  tiles int32 [n, 4] = (row0, rows <= max_rows, pos0, slot) -> [T, heads*vdim].
@@ -822,9 +834,12 @@ def paged_attention(q: torch.Tensor, pool: torch.Tensor, page_tables: torch.Tens
     window > 0: a key is seen only when it is less than `window` positions back or among the first `keep_first`
     of its sequence.  talk_after: talk mixes the heads' softmax weights instead of their scores (no sink then).
     head_scale fp32 [heads]: per-head multiplier of the scores.  softcap > 0: every head's own scaled score becomes
-    softcap * tanh(score / softcap) before mixing, bias and softmax."""
-    assert q.dtype == torch.float32 and q.is_contiguous() and q.shape[1] == heads * dim
-    assert pool.dim() == 2 and pool.is_contiguous() and pool.shape[1] == kv_heads * (dim + vdim)
+    softcap * tanh(score / softcap) before mixing, bias and softmax.
+    diff = (lambda, scale, eps): differential attention.  q [T, heads*2*dim], pool rows k (kv_heads*2*dim) | v (kv_heads*vdim),
+    two maps a1, a2 per head over the same values, out = rms(a1 - lambda a2) * scale per head (eps inside the root), gated."""
+    maps = 1 if diff is None else 2
+    assert q.dtype == torch.float32 and q.is_contiguous() and q.shape[1] == heads * maps * dim
+    assert pool.dim() == 2 and pool.is_contiguous() and pool.shape[1] == kv_heads * (maps * dim + vdim)
     if out is None:
         out = torch.empty(q.shape[0], heads * vdim, dtype=out_dtype or pool.dtype, device=q.device)
     assert out.shape == (q.shape[0], heads * vdim) and out.is_contiguous()
@@ -849,11 +864,13 @@ def paged_attention(q: torch.Tensor, pool: torch.Tensor, page_tables: torch.Tens
     if head_scale is not None:
         assert head_scale.numel() == heads
         p.head_scale = _f32(head_scale, "head_scale")
-    p.softcap = float(softcap)
+    p.softcap, p.maps = float(softcap), maps
+    if diff is not None:
+        p.diff_lambda, p.diff_scale, p.diff_eps = (float(v) for v in diff)
     p.nsplit = max(1, int(nsplit)) if max_rows == 1 else 1
     partial = None
     if p.nsplit > 1:
-        partial = torch.empty(q.shape[0] * p.nsplit * heads * (vdim + 2), dtype=torch.float32, device=q.device)
+        partial = torch.empty(q.shape[0] * p.nsplit * heads * maps * (vdim + 2), dtype=torch.float32, device=q.device)
         p.partial = partial.data_ptr()
     check(_lib.load().vila_paged_attention(C.byref(p), _stream()), "vila_paged_attention")
     return out
@@ -873,6 +890,34 @@ def moe_route_sigmoid(x: torch.Tensor, w_router: torch.Tensor, correction: Optio
                                              _f32(correction, "correction"), _p(idx), _p(wt), rows, cols, E, top,
                                              groups, keep, _stream()), "vila_moe_route_sigmoid")
     return idx, wt
+
+
+SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
+
+
+def moe_route_scores(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], top: int, *,
+                     score: int = SCORE_SIGMOID, groups: int = 1, keep: int = 1, group_top: int = 2, scale: float = 1.0,
+                     gate_w: Optional[torch.Tensor] = None):
+    """Router with sigmoid or softmax scores over all of w_router's outputs and group-limited choice -> (idx int32
+    [rows, top], weight fp32 [rows, top], gate fp32 [rows] or None): choice = score + correction, restricted to the `keep`
+    groups (of `groups`) with the best largest choice value (group_top 1) or sum of their two largest (2); weights are
+    scale * the plain scores.  gate_w fp32 [cols]: also gate = sigmoid(x . gate_w)."""
+    assert x.dim() == 2 and x.stride(1) == 1 and w_router.shape[1] == x.shape[1]
+    rows, cols = x.shape
+    E = w_router.shape[0]
+    idx = torch.empty(rows, top, dtype=torch.int32, device=x.device)
+    wt = torch.empty(rows, top, dtype=torch.float32, device=x.device)
+    gate = torch.empty(rows, dtype=torch.float32, device=x.device) if gate_w is not None else None
+    p = _lib.MoeRouteParams()
+    p.x, p.ldx, p.x_dtype, p.w = _p(x), x.stride(0), _dt(x, "x"), _f32(w_router, "w_router")
+    assert correction is None or correction.numel() == E
+    assert gate_w is None or gate_w.numel() == cols
+    p.correction, p.gate_w = _f32(correction, "correction"), _f32(gate_w, "gate_w")
+    p.idx, p.weight, p.gate = _p(idx), _p(wt), _p(gate)
+    p.rows, p.cols, p.experts, p.top, p.groups, p.keep = rows, cols, E, top, groups, keep
+    p.score, p.group_top, p.scale = score, group_top, float(scale)
+    check(_lib.load().vila_moe_route_scores(C.byref(p), _stream()), "vila_moe_route_scores")
+    return idx, wt, gate
 
 
 def residual_add_rows(x: torch.Tensor, a: Optional[torch.Tensor] = None, part: Optional[torch.Tensor] = None, *,
@@ -1095,16 +1140,87 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
     return out
 
 
-def gated_head_norm_rows(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, *, heads: int, eps: float, out_dtype=None
-                         ) -> torch.Tensor:
-    """o fp32 [T, heads*vdim] -> rms(o per head) * w [vdim] * silu(gate [T, heads*vdim]) (gate: a view is fine)"""
+def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, *, heads: int, dim: int,
+               vdim: int, decay: torch.Tensor, silu: bool = False, q_scale: float = 1.0) -> torch.Tensor:
+    """Linear attention with one constant decay per head: S <- decay S + k v^T, o = S^T (q_scale q); silu: q, k and v are
+    pre-activations.  q, k [T, heads*dim], v [T, heads*vdim] (views with a row stride are fine, one dtype); decay fp32
+    [heads]; state fp32 [slots, heads, vdim, dim], advanced in place; seqs int32 [n, 4] -> o fp32 [T, heads*vdim]."""
+    T = q.shape[0]
+    assert q.shape == k.shape == (T, heads * dim) and v.shape == (T, heads * vdim)
+    assert q.stride(1) == k.stride(1) == v.stride(1) == 1 and q.dtype == k.dtype == v.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, vdim, dim)
+    assert decay.numel() == heads
+    out = torch.empty(T, heads * vdim, dtype=torch.float32, device=q.device)
+    p = _lib.DecayScanParams()
+    p.q, p.k, p.v, p.ld_q, p.ld_k, p.ld_v = _p(q), _p(k), _p(v), q.stride(0), k.stride(0), v.stride(0)
+    p.decay = _f32(decay, "decay")
+    p.state, p.seqs, p.out, p.ld_out = _p(state), _i32(seqs, "seqs"), _p(out), out.stride(0)
+    p.in_dtype, p.nseq, p.H, p.dim, p.vdim, p.silu, p.q_scale = _dt(q, "q"), seqs.shape[0], heads, dim, vdim, 1 if silu else 0, q_scale
+    check(_lib.load().vila_decay_scan(C.byref(p), _stream()), "vila_decay_scan")
+    return out
+
+
+def gated_head_norm_rows(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, *, heads: int, eps: float, out_dtype=None,
+                         gate_act: int = ACT_SILU) -> torch.Tensor:
+    """o fp32 [T, heads*vdim] -> rms(o per head) * w [vdim] * act(gate [T, heads*vdim]) (gate: a view is fine; act: SiLU or
+    ACT_SIGMOID; heads = 1: one norm over the whole row)"""
     assert o.dtype == torch.float32 and o.is_contiguous() and o.dim() == 2 and o.shape[1] % heads == 0
     T, vdim = o.shape[0], o.shape[1] // heads
     assert w.numel() == vdim and gate.shape == o.shape and gate.stride(1) == 1
     out = torch.empty(o.shape, dtype=out_dtype or gate.dtype, device=o.device)
-    check(_lib.load().vila_gated_head_norm_rows(_p(o), _f32(w, "w"), _p(gate), _dt(gate, "gate"), gate.stride(0), eps, _p(out),
-                                                _dt(out, "out"), T, heads, vdim, _stream()), "vila_gated_head_norm_rows")
+    check(_lib.load().vila_gated_head_norm_act_rows(_p(o), _f32(w, "w"), _p(gate), _dt(gate, "gate"), gate.stride(0), eps, _p(out),
+                                                    _dt(out, "out"), T, heads, vdim, gate_act, _stream()),
+          "vila_gated_head_norm_act_rows")
     return out
+
+
+class TanhNorm:
+    """A Dynamic Tanh norm: tanh(alpha x) * w + bias, alpha a number, w and bias fp32 [cols]"""
+
+    def __init__(self, alpha: float, w: torch.Tensor, bias: torch.Tensor):
+        self.alpha, self.w, self.bias = float(alpha), w, bias
+
+
+def tanh_residual_rows(x: torch.Tensor, norms: Sequence[TanhNorm], *, out_dtype, a: Optional[torch.Tensor] = None,
+                       a_scale: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None,
+                       b_scale: Optional[torch.Tensor] = None, b_gate: Optional[torch.Tensor] = None,
+                       part: Optional[torch.Tensor] = None, n_partials: int = 1, idx: Optional[torch.Tensor] = None,
+                       weight: Optional[torch.Tensor] = None, experts: int = 0, h: Optional[torch.Tensor] = None,
+                       mult: float = 1.0, table: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None):
+    """x fp32 [rows, cols] (in place) += mult * (a_scale * a + b_scale * f), f = b * b_gate + sum_j partial j, then up to two
+    Dynamic Tanh norms of the result -> list of [rows, cols] in out_dtype.  Partial j of row r is part[r * n_partials + j],
+    or, for idx[r, j] >= experts (an identity expert), weight[r, j] * h[r].  table / ids: x starts as the embedding rows
+    table[ids] instead of its content."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2 and len(norms) <= 2
+    rows, cols = x.shape
+    p = _lib.TanhResidualParams()
+    p.x, p.rows, p.cols, p.mult, p.n_out = _p(x), rows, cols, float(mult), len(norms)
+    if table is not None:
+        assert table.is_contiguous() and table.shape[1] == cols and ids.numel() == rows
+        p.table, p.table_dtype, p.ids = _p(table), _dt(table, "table"), _i32(ids, "ids")
+    if a is not None:
+        assert a.shape == (rows, cols) and a.stride(1) == 1 and a_scale.numel() == cols
+        p.a, p.lda, p.a_dtype, p.a_scale = _p(a), a.stride(0), _dt(a, "a"), _f32(a_scale, "a_scale")
+    if b is not None or part is not None:
+        assert a is not None and b_scale.numel() == cols
+        p.b_scale = _f32(b_scale, "b_scale")
+    if b is not None:
+        assert b.shape == (rows, cols) and b.stride(1) == 1 and (b_gate is None or b_gate.numel() == rows)
+        p.b, p.ldb, p.b_dtype, p.b_gate = _p(b), b.stride(0), _dt(b, "b"), _f32(b_gate, "b_gate")
+    if part is not None:
+        assert part.shape == (rows * n_partials, cols) and part.stride(1) == 1
+        p.part, p.ldp, p.part_dtype, p.n_partials = _p(part), part.stride(0), _dt(part, "part"), n_partials
+        if idx is not None:
+            assert idx.numel() == weight.numel() == rows * n_partials and h.shape == (rows, cols) and h.stride(1) == 1
+            p.idx, p.weight, p.experts = _i32(idx, "idx"), _f32(weight, "weight"), experts
+            p.h, p.ldh, p.h_dtype = _p(h), h.stride(0), _dt(h, "h")
+    outs = [torch.empty(rows, cols, dtype=out_dtype, device=x.device) for _ in norms]
+    for k, n in enumerate(norms):
+        assert n.w.numel() == n.bias.numel() == cols
+        p.w[k], p.bias[k], p.alpha[k] = _f32(n.w, "w"), _f32(n.bias, "bias"), n.alpha
+        p.out[k], p.out_dtype = _p(outs[k]), _dt(outs[k], "out")
+    check(_lib.load().vila_tanh_residual_rows(C.byref(p), _stream()), "vila_tanh_residual_rows")
+    return outs
 
 
 def scaled_residual_norm_rows(x: torch.Tensor, a: torch.Tensor, a_scale: torch.Tensor, b: Optional[torch.Tensor] = None,
