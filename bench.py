@@ -2090,6 +2090,264 @@ def run_delta_lm(args):
     print(json.dumps(res))
 
 
+# ------------------------------------------------------------------------------------------------
+# --workload lightning_lm: the Nibelix language model (lightning attention, windowed differential attention, Dynamic Tanh
+# norms, routed experts with identity experts and a gated shared expert, parallel sublayers) next to the two models of the
+# package that are closest to its halves, at equal width / heads / vocabulary, random weights, bf16: Bivizen (recurrent and
+# attention mixers with parallel sublayers, dense feed-forwards) and Lufatar (attention with routed experts in parallel).
+# The ledger sets every kernel beside the like kernel of those two and of Ludazen (windowed attention).
+# ------------------------------------------------------------------------------------------------
+LIGHTNING_LM = dict(window=1024)
+
+
+def lightning_lm_config(z):
+    W, H, G = z["width"], z["heads"], z["kv_heads"]
+    lig = {"decay": [1.0 - 2.0 ** (-1.0 - 9.0 * i / H) for i in range(H)], "dim": 128, "heads": H, "vdim": 128}
+    att = {"diff": 0.4, "dim": 64, "heads": H, "kv_heads": G, "mask": {"size": LIGHTNING_LM["window"]},
+           "rot": {"base": 10000.0, "dims": 64}, "scale": 0.125, "vdim": 128}
+    dense = {"ff": W * 8 // 3 // 64 * 64, "kind": "dense"}
+    moe = {"expert": {"ff": z["expert_ff"]}, "kind": "moe", "shared": {"ff": z["expert_ff"]},
+           "router": {"experts": z["experts"] - 4, "groups": {"count": 4, "keep": 2}, "identity": 4, "scale": 2.0, "top": z["top"]}}
+    return {"architecture": "Nibelix", "layers": [{"type": t, "mixer": dict(m), "mlp": dict(f)} for t, m, f in (
+        ("lightning", lig, dense), ("attention", att, moe), ("lightning", lig, moe), ("attention", att, dense))],
+        "logit_softcap": 30.0, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "vocab": z["vocab"], "width": W}
+
+
+def lightning_lm_twin(z):
+    """Bivizen with the same mixers' sizes: gla, attention, gla, attention"""
+    d = delta_lm_config(dict(z, ff=4 * z["width"]))
+    att, gla = d["layers"][0], d["layers"][1]
+    return dict(d, layers=[gla, att, gla, att])
+
+
+def lightning_lm_block(args, peaks):
+    import torch
+
+    from vila_b200 import ops
+    from vila_b200.model import (BivizenConfig, BivizenForCausalLM, LufatarConfig, LufatarForCausalLM, NibelixConfig,
+                                 NibelixForCausalLM)
+    from vila_b200.serving import TokenEngine
+    dev = torch.device("cuda:0")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+
+    def timed(fn, reps=args.steps, warm=max(3, args.warmup), setup=None):
+        ts = []
+        for i in range(warm + reps):
+            if setup is not None:
+                setup()
+            flush.fill_(i & 255)     # evict L2 (126 MB) between iterations
+            a, b = ev(), ev()
+            torch.cuda.synchronize()
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            if i >= warm:
+                ts.append(a.elapsed_time(b))
+        ts.sort()
+        return ts[len(ts) // 2]
+
+    def timed_op(fn):
+        """captured once, timed as a graph replay: the device time of the op's launches, not the host time around them"""
+        fn()
+        fn()
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            fn()
+        return timed(g.replay)
+
+    S, B, CTX, NEW = 2048, 8, 1024, 32
+    tf, gbs = peaks["bf16_tflops"], peaks["hbm_gbs"]
+    bf = torch.bfloat16
+    out = {}
+    t00 = time.time()
+
+    def log(msg):
+        print("[lightning_lm %6.1fs] %s" % (time.time() - t00, msg), file=sys.stderr, flush=True)
+
+    def engine_numbers(lm, prompt):
+        eng = TokenEngine(lm, max_tokens=B * (CTX + 4 * NEW + 64), slots=B)
+        t_pre = timed(lambda: eng.step([("p", prompt, [S - 1])]), setup=lambda: eng.release("p"))
+        eng.release("p")
+        for b in range(B):
+            eng.step([(b, prompt[:CTX], [])])
+        step_in = [[(b, [int(prompt[(k * 7 + b) % S])], [0]) for b in range(B)] for k in range(NEW)]
+
+        def decode_run():
+            for k in range(NEW):
+                eng.step(step_in[k])
+        t_dec = timed(decode_run, reps=3, warm=1)     # contexts grow CTX .. CTX + 4 * NEW: fits the reserve
+        for b in range(B):
+            eng.release(b)
+        n = sum(v.numel() for v in lm.weights.values())
+        return eng, {"params_m": n / 1e6, "prefill_tok_s": S / t_pre * 1e3, "prefill_ms": t_pre,
+                     "decode_tok_s": B * NEW / t_dec * 1e3, "decode_ms_per_step": t_dec / NEW}
+
+    def flops(t, fl):
+        return {"ms": t, "tflops": fl / t / 1e9, "of_bf16_peak": fl / t / 1e9 / tf}
+
+    def bytes_(t, by):
+        return {"ms": t, "gbs": by / t / 1e6, "of_hbm": by / t / 1e6 / gbs}
+
+    for name, z in PARALLEL_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        W, H, G = z["width"], z["heads"], z["kv_heads"]
+        g = torch.Generator().manual_seed(0)
+        prompt = torch.randint(0, z["vocab"], (S,), generator=g).tolist()
+        log("size %s: nibelix" % name)
+        lm = NibelixForCausalLM(NibelixConfig.from_dict(lightning_lm_config(z)), dev, bf).init_random(0, on_device=True)
+        eng, res_new = engine_numbers(lm, prompt)
+        log("size %s: bivizen" % name)
+        tw = BivizenForCausalLM(BivizenConfig.from_dict(lightning_lm_twin(z)), dev, bf).init_random(0, on_device=True)
+        eng2, res_biv = engine_numbers(tw, prompt)
+        log("size %s: lufatar" % name)
+        tl = LufatarForCausalLM(LufatarConfig.from_dict(parallel_lm_config(z)), dev, bf).init_random(0, on_device=True)
+        eng3, res_luf = engine_numbers(tl, prompt)
+        # ---- kernel beside the like kernel ---------------------------------------------------------------
+        log("kernel ledger")
+        led = {}
+        Ll, La, Lb, T0 = lm.layers[0], lm.layers[1], tw.layers[0], tl.layers[0]
+        D = 128
+        # scans over states [H, 128, 128]: flops counted as 2 per multiply-add of the recurrence's own products
+        sq1 = torch.tensor([[0, S, 0, 0]], dtype=torch.int32, device=dev)
+        sqB = torch.tensor([(b, 1, CTX, b) for b in range(B)], dtype=torch.int32, device=dev)
+        sqP = torch.tensor([(b * (S // B), S // B, 0, b) for b in range(B)], dtype=torch.int32, device=dev)
+        std, stg = eng.cache.state[(0, "scan")], eng2.cache.state[(0, "scan")]
+        wide = (torch.randn(S, 4 * H * D + 8, device=dev) * 0.5).to(bf)
+        for rows, sq, tag in ((S, sq1, "prefill, one %d-row prompt" % S), (S, sqP, "prefill, %d prompts of %d rows" % (B, S // B)),
+                              (B, sqB, "decode, %d rows" % B)):
+            nseq = sq.shape[0]
+            x = wide[:rows]
+            q, k, v, zz = (x[:, i * H * D:(i + 1) * H * D] for i in range(4))
+            rate = (lambda t, fl, by: bytes_(t, by)) if rows == B else (lambda t, fl, by: {"ms": t, "tflops_fp32": fl / t / 1e9})
+            st_by = 2 * nseq * H * D * D * 4
+            t = timed_op(lambda: ops.decay_scan(q, k, v, std, sq, heads=H, dim=D, vdim=D, decay=Ll.decay, silu=True))
+            led["decay_scan with SiLU on q, k, v " + tag] = rate(t, 6.0 * rows * H * D * D, st_by + rows * H * D * (6 + 4))
+            t = timed_op(lambda: ops.gla_scan(q, k, v, zz, stg, sq, heads=H, dim=D, vdim=D, q_scale=D ** -0.5, tau=8.0, z_bias=Lb.a2_b))
+            led["bivizen gla_scan, the same state " + tag] = rate(t, 6.0 * rows * H * D * D, st_by + rows * H * D * (8 + 4))
+        # attention: two maps of 64 columns, window; beside one map of 128 columns with Ludazen's window and with none
+        page, npg = eng.cache.page, eng.cache.n_pages
+        win = LIGHTNING_LM["window"]
+        pool, pool1 = eng.cache.latent[1], eng2.cache.latent[1]
+        pt = torch.arange(npg, dtype=torch.int32, device=dev).view(1, -1).repeat(B, 1).contiguous()
+        tiles = torch.tensor([(o, 16, o, 0) for o in range(0, S, 16)], dtype=torch.int32, device=dev)
+        q = torch.randn(S, H * 2 * 64, device=dev)
+        gate = torch.randn(S, H, device=dev).to(bf)
+        akw = dict(heads=H, kv_heads=G, vdim=D, page=page, scale=0.1)
+        pairs_w = sum(min(p + 1, win) for p in range(S))
+        # two maps: 2 * 64 multiply-adds of scores, 2 * 128 of values per (query, key) pair and head; one map: 128 + 128
+        att = lambda t, pairs, per: {"ms": t, "tflops_fp32": H * pairs * per / t / 1e9}
+        t = timed_op(lambda: ops.paged_attention(q, pool, pt, tiles, max_rows=16, dim=64, window=win, diff=La.diff, gate=gate, **akw))
+        led["paged_attention prefill: two maps, window %d, combined, gate" % win] = att(t, pairs_w, 2.0 * (2 * 64 + 2 * D))
+        t = timed_op(lambda: ops.paged_attention(q, pool1, pt, tiles, max_rows=16, dim=D, window=win, gate=gate, **akw))
+        led["paged_attention prefill: one map, window %d, gate" % win] = att(t, pairs_w, 2.0 * (D + D))
+        t = timed_op(lambda: ops.paged_attention(q, pool1, pt, tiles, max_rows=16, dim=D, softcap=30.0, gate=gate, **akw))
+        led["bivizen paged_attention prefill: one map, causal, cap, gate"] = att(t, S * (S + 1) / 2, 2.0 * (D + D))
+        dt_ = torch.tensor([(b, 1, CTX - 1, b) for b in range(B)], dtype=torch.int32, device=dev)
+        pt2 = ((torch.arange(B, device=dev, dtype=torch.int32)[:, None] * (CTX // page) +
+                torch.arange(npg, device=dev, dtype=torch.int32)[None]) % npg).contiguous()
+        ns = eng.cache.decode_splits
+        t = timed_op(lambda: ops.paged_attention(q[:B], pool, pt2, dt_, max_rows=1, nsplit=ns, dim=64, window=win, diff=La.diff,
+                                                 gate=gate[:B], **akw))
+        led["paged_attention decode: two maps, window, combined, gate (8 x 1024 keys)"] = bytes_(t, B * CTX * G * (2 * 64 + D) * 2)
+        t = timed_op(lambda: ops.paged_attention(q[:B], pool1, pt2, dt_, max_rows=1, nsplit=ns, dim=D, softcap=30.0, gate=gate[:B], **akw))
+        led["bivizen paged_attention decode: one map, cap, gate (8 x 1024 keys)"] = bytes_(t, B * CTX * G * 2 * D * 2)
+        ar = torch.arange(S, dtype=torch.int32, device=dev)
+        qkv = wide[:, :(H + 2 * G) * D]
+        by = S * ((H + 2 * G) * D * 2 + H * D * 4 + 2 * G * D * 2)
+        t = timed_op(lambda: ops.rope_append(qkv, ar, ar, pool, heads=H, kv_heads=G, dim=64, vdim=D, inv_freq=La.inv_freq,
+                                             unit_norm=False, eps=0.0, halves=True, maps=2))
+        led["rope_append: two maps + k | v append (2048 rows)"] = bytes_(t, by)
+        t = timed_op(lambda: ops.rope_append(qkv, ar, ar, pool1, heads=H, kv_heads=G, dim=D, vdim=D, inv_freq=tw.layers[1].inv_freq,
+                                             unit_norm=False, eps=0.0, halves=True))
+        led["bivizen rope_append: one map (2048 rows)"] = bytes_(t, by)
+        # row kernels
+        x = torch.randn(S, W, device=dev)
+        y1, y2 = torch.randn(S, W, device=dev).to(bf), torch.randn(S, W, device=dev).to(bf)
+        o = torch.randn(S, H * D, device=dev)
+        gt = wide[:, :H * D]
+        for rows, tag in ((S, "2048 rows"), (B, "decode, 8 rows")):
+            by = rows * H * D * (4 + 2 + 2)
+            t = timed_op(lambda: ops.gated_head_norm_rows(o[:rows], Ll.norm, gt[:rows], heads=1, eps=1e-5, out_dtype=bf, gate_act=ops.ACT_SIGMOID))
+            led["gated_head_norm_rows: one norm over all heads, sigmoid gate (%s)" % tag] = bytes_(t, by)
+            t = timed_op(lambda: ops.gated_head_norm_rows(o[:rows], Lb.norm, gt[:rows], heads=H, eps=1e-5, out_dtype=bf))
+            led["bivizen gated_head_norm_rows: per head, SiLU gate (%s)" % tag] = bytes_(t, by)
+            t = timed_op(lambda: ops.tanh_residual_rows(x[:rows], lm.layers[1].norms, out_dtype=bf, a=y1[:rows], a_scale=Ll.ls1, b=y2[:rows],
+                                                        b_scale=Ll.ls2, mult=0.5))
+            led["tanh_residual_rows: two branches, two norms (%s)" % tag] = bytes_(t, rows * W * (8 + 2 + 2 + 4))
+            t = timed_op(lambda: ops.scaled_residual_norm_rows(x[:rows], y1[:rows], Lb.ls1, y2[:rows], Lb.ls2, Lb.norm1, 1e-5, out_dtype=bf))
+            led["bivizen scaled_residual_norm_rows: two branches, one norm (%s)" % tag] = bytes_(t, rows * W * (8 + 2 + 2 + 2))
+        hb = torch.randn(S, W, device=dev).to(bf)
+        top, E = z["top"], z["experts"]
+        idx, wt, sg = ops.moe_route_scores(hb, La.router, La.correction, top, score=ops.SCORE_SOFTMAX, groups=4, keep=2, group_top=1,
+                                           scale=2.0, gate_w=La.shared_gate)
+        pf = torch.randn(S * top, W, device=dev)
+        t = timed_op(lambda: ops.tanh_residual_rows(x, lm.layers[2].norms, out_dtype=bf, a=y1, a_scale=La.ls1, b=y2, b_scale=La.ls2, b_gate=sg,
+                                                    part=pf, n_partials=top, idx=idx, weight=wt, experts=E - 4, h=hb, mult=0.5))
+        led["tanh_residual_rows: gated shared + %d routed partials, two norms (2048 rows)" % top] = bytes_(t, S * W * (8 + 2 + 2 + 4 + 4 * top))
+        t = timed_op(lambda: ops.residual_norm_rows(x, y1, La.ls1, 1e-5, part=pf, n_partials=top, out_dtype=bf))
+        led["ludazen residual_norm_rows: %d partials, one norm (2048 rows)" % top] = bytes_(t, S * W * (8 + 2 + 2 + 4 * top))
+        # router and experts
+        for rows, tag in ((S, "2048 rows"), (B, "decode, 8 rows")):
+            by = rows * W * 2 + E * W * 4
+            t = timed_op(lambda: ops.moe_route_scores(hb[:rows], La.router, La.correction, top, score=ops.SCORE_SOFTMAX, groups=4, keep=2,
+                                                      group_top=1, scale=2.0, gate_w=La.shared_gate))
+            led["moe_route_scores: softmax, largest of the group, shared gate (%s)" % tag] = bytes_(t, by)
+            t = timed_op(lambda: ops.moe_route_sigmoid(hb[:rows], T0.router, T0.correction, top, 4, 2))
+            led["lufatar moe_route_sigmoid (%s)" % tag] = bytes_(t, by)
+        real = float((idx < E - 4).float().mean())     # share of choices that are experts with tensors
+        fe = z["expert_ff"]
+        t = timed_op(lambda: lm._experts(La, hb))
+        led["routed + shared experts prefill"] = dict(flops(t, 2.0 * S * W * fe * 2 * (top * real + 1)), routed_share=real)
+        t = timed_op(lambda: tl._experts(T0, hb))
+        led["lufatar routed experts prefill"] = flops(t, 2.0 * S * W * fe * 3 * top)
+        hit = len(set(i for i in idx[:B].reshape(-1).tolist() if i < E - 4))
+        t = timed_op(lambda: lm._experts(La, hb[:B]))
+        led["routed + shared experts decode (8 rows)"] = dict(bytes_(t, 2 * (hit + 1) * fe * W * 2 + E * W * 4), experts_hit=hit)
+        hl = len(set(ops.moe_route_sigmoid(hb[:B], T0.router, T0.correction, top, 4, 2)[0].reshape(-1).tolist()))
+        t = timed_op(lambda: tl._experts(T0, hb[:B]))
+        led["lufatar routed experts decode (8 rows)"] = dict(bytes_(t, 3 * hl * fe * W * 2 + E * W * 4), experts_hit=hl)
+        # projections
+        fl = 2.0 * S * W * Ll.gu.shape[0]
+        for tag, kw in (("gelu-gated", dict(geglu=True)), ("bivizen clamped", dict(glu_clamp=(1.702, 7.0))), ("SwiGLU", dict(swiglu=True))):
+            t = timed_op(lambda: ops.linear_any(hb, Ll.gu, **kw))
+            led["gate | up projection, %s epilogue (tcgen05)" % tag] = flops(t, fl)
+            t = timed_op(lambda: ops.linear_any(hb[:B], Ll.gu, **kw))
+            led["gate | up projection decode, %s epilogue (8 rows)" % tag] = bytes_(t, Ll.gu.numel() * 2)
+        hx = x[:B].contiguous()
+        t = timed_op(lambda: lm.logits(hx))
+        led["final norm + head + cap (8 rows)"] = bytes_(t, lm.head.numel() * 2)
+        t = timed_op(lambda: tw.logits(hx))
+        led["bivizen final norm + head (8 rows)"] = bytes_(t, tw.head.numel() * 2)
+        out[name] = {"nibelix": res_new, "bivizen": res_biv, "lufatar": res_luf, "kernels": led}
+        del lm, tw, tl, eng, eng2, eng3
+        torch.cuda.empty_cache()
+    return {"workload": "lightning_lm: 4 Nibelix layers (lightning + dense; windowed differential attention + routed experts; lightning + "
+                        "routed experts; differential attention + dense) vs 4 Bivizen layers (gated linear attention, capped attention, twice; "
+                        "dense) and 4 Lufatar layers (attention + routed experts) of equal width / heads / vocabulary / experts; prefill: one "
+                        "%d-token prompt; decode: %d sequences x %d-token context, %d steps" % (S, B, CTX, NEW),
+            "dtype": "bf16", "data": "synthetic (random weights, random ids)",
+            "l2_policy": "256 MB buffer written between timed iterations",
+            "kernel_ledger_timing": "each op captured in a CUDA graph, one replay per timed iteration", "peaks": peaks, "sizes": out}
+
+
+def run_lightning_lm(args):
+    import torch
+    assert torch.cuda.is_available(), "bench.py --workload lightning_lm needs a GPU"
+    import faulthandler
+    faulthandler.dump_traceback_later(int(os.environ.get("VILA_BENCH_WATCHDOG_S", "480")), exit=True)
+    peaks = read_peaks()
+    with ClockSampler(0) as cs:
+        res = lightning_lm_block(args, peaks)
+    res["clocks"] = cs.summary()
+    from vila_b200 import _lib
+    res["gpu_launches"] = _lib.LAUNCHES
+    print(json.dumps(res))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -2104,12 +2362,13 @@ def main():
     ap.add_argument("--sp-steps", type=int, default=10)
     ap.add_argument("--profile", action="store_true",
                     help="profiling aid (ncu): 1 warm-up, 8 new tokens, no extra blocks; NOT a valid bench number")
-    ap.add_argument("--sizes", default="", help="hybrid_lm / parallel_lm / ssm_lm / window_lm / delta_lm: comma-separated subset of the workload's sizes ("
+    ap.add_argument("--sizes", default="", help="hybrid_lm / parallel_lm / ssm_lm / window_lm / delta_lm / lightning_lm: comma-separated subset of the workload's sizes ("
                     + ",".join(HYBRID_SIZES) + " / " + ",".join(PARALLEL_SIZES) + ")")
-    ap.add_argument("--workload", default="headline", choices=["headline", "hybrid_lm", "parallel_lm", "ssm_lm", "window_lm", "delta_lm"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "hybrid_lm", "parallel_lm", "ssm_lm", "window_lm", "delta_lm", "lightning_lm"],
                     help="headline (default): the NVILA-8B serving step; hybrid_lm: Moronex vs Qwen2 at equal size; "
                          "parallel_lm: Lufatar vs Moronex at equal size; ssm_lm: Nusovik vs Moronex at equal size; "
-                         "window_lm: Ludazen vs Lufatar at equal size; delta_lm: Bivizen vs Nusovik at equal size")
+                         "window_lm: Ludazen vs Lufatar at equal size; delta_lm: Bivizen vs Nusovik at equal size; "
+                         "lightning_lm: Nibelix vs Bivizen and Lufatar at equal size")
     args = ap.parse_args()
     if args.workload == "hybrid_lm":
         return run_hybrid_lm(args)
@@ -2121,6 +2380,8 @@ def main():
         return run_window_lm(args)
     if args.workload == "delta_lm":
         return run_delta_lm(args)
+    if args.workload == "lightning_lm":
+        return run_lightning_lm(args)
     if args.profile:
         global NEW_TOKENS
         NEW_TOKENS = 8
