@@ -54,7 +54,6 @@ struct SkinnyArgs {
   float* ws;        // [n_blk][split][m_pad][128] fp32 partials
   int* counters;    // [n_blocks]
   GemmEpilogue epi;
-  int dbg_skip;     // profiling aid: 1 = skip the global stores, 2 = skip the transposed read-out
   long long* dbg;   // profiling aid (VILA_B200_GEMM_DEBUG): 16 counters per CTA, or nullptr
 };
 
@@ -117,7 +116,7 @@ __device__ __forceinline__ void readout(const uint8_t* buf, int epi_tid, int c, 
   for (int i = 0; i < kIters; ++i) {
     const int q = epi_tid + i * 128;
     const int m = c * 32 + q / kVpr, nn = nc0 + (q % kVpr) * 8;
-    if (m < a.M && nn < n_out && a.dbg_skip != 1) stg_v4(a.C + static_cast<size_t>(m) * a.ldc + nn, o[i]);
+    if (m < a.M && nn < n_out) stg_v4(a.C + static_cast<size_t>(m) * a.ldc + nn, o[i]);
   }
 }
 
@@ -479,11 +478,9 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
       }
       epi_group_sync(wg);
       // transposed read-out: 16-byte vectors along the feature dimension
-      if (a.dbg_skip != 2) {
-        if (a.epi.rope_table != nullptr) readout_rope(buf, epi_tid, c, n_blk, a);
-        else if (swiglu) readout<8>(buf, epi_tid, c, nc0, n_out, a);
-        else readout<16>(buf, epi_tid, c, nc0, n_out, a);
-      }
+      if (a.epi.rope_table != nullptr) readout_rope(buf, epi_tid, c, n_blk, a);
+      else if (swiglu) readout<8>(buf, epi_tid, c, nc0, n_out, a);
+      else readout<16>(buf, epi_tid, c, nc0, n_out, a);
       epi_group_sync(wg);  // the staging tile may be overwritten
     }
   }
@@ -593,10 +590,8 @@ int launch_skinny(const __nv_bfloat16* A, int lda, const __nv_bfloat16* W, int l
   a.ws = ws_ptr ? reinterpret_cast<float*>(static_cast<char*>(ws_ptr) + kCounterBytes) : nullptr;
   a.epi = epi;
   a.dbg = nullptr;
-  a.dbg_skip = 0;
 #ifdef VILA_B200_DEBUG_HOOKS  // profiling aids, compiled OUT of the shipped library (an env var
                               // must not be able to make a kernel write through an arbitrary pointer)
-  if (const char* e = getenv("VILA_B200_GEMM_DEBUG_SKIP")) a.dbg_skip = atoi(e);
   if (const char* e = getenv("VILA_B200_GEMM_DEBUG")) {  // hex device pointer (tools/skinny_phase_times.py)
     unsigned long long ptr = 0;
     if (sscanf(e, "%llx", &ptr) == 1) a.dbg = reinterpret_cast<long long*>(ptr);
