@@ -2199,6 +2199,9 @@ def lightning_lm_block(args, peaks):
         prompt = torch.randint(0, z["vocab"], (S,), generator=g).tolist()
         log("size %s: nibelix" % name)
         lm = NibelixForCausalLM(NibelixConfig.from_dict(lightning_lm_config(z)), dev, bf).init_random(0, on_device=True)
+        for L in lm.layers:          # random corrections would outweigh the scores and send all tokens to the same experts
+            if L.cfg.mlp_kind == "moe":
+                L.correction.zero_()
         eng, res_new = engine_numbers(lm, prompt)
         log("size %s: bivizen" % name)
         tw = BivizenForCausalLM(BivizenConfig.from_dict(lightning_lm_twin(z)), dev, bf).init_random(0, on_device=True)

@@ -178,22 +178,69 @@ __device__ __forceinline__ float out_gate(const vila_paged_attn_params& p, int r
   return p.gate ? sigmoid_f(ld_any(p.gate, p.gate_dtype, static_cast<size_t>(row) * p.ldg + h)) : 1.0f;
 }
 
-// K | V rows of a key block, widened to fp32: one warp per key.  16-byte loads when the head sizes allow
-// (bf16: multiples of 8, fp32: multiples of 4; the pool row is then 16-byte aligned as well).
-// g0, G: the value heads g0 .. g0 + G - 1 of the pool row are loaded (all of them by default) with their key heads (as
-// many, or one per map).
-__device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_paged_attn_params& p,
-                                              const int32_t* pt, int j0, int nkeys, int BK, int D4, int DS, int V4,
-                                              int nwarps = kWarps, int g0 = 0, int G = 0, bool with_v = true) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (G == 0) G = p.G;
-  const int maps = maps_of(p.maps), GK = G * maps;
-  const int D = p.dim, V = p.vdim, KS = key_stride(GK, DS);
+// K | V rows of a key block, widened to fp32.  16-byte loads when the head sizes allow (bf16: multiples of 8, fp32:
+// multiples of 4; the pool row is then 16-byte aligned as well): the block's pieces are dealt to all threads, and a thread
+// has kLoads of them in flight before it stores the first.  Otherwise a warp per key, element by element.
+// g0, G: the value heads g0 .. g0 + G - 1 of the pool row are loaded with their key heads (as many, or one per map).
+constexpr int kLoads = 4;
+
+template <bool BF16>
+__device__ __forceinline__ void load_kv_vec(float* Ks, float* Vs, const vila_paged_attn_params& p, const int32_t* pt, int j0,
+                                            int nkeys, int BK, int DS, int V4, int nthreads, int g0, int G, bool with_v) {
+  constexpr int E = BF16 ? 8 : 4;   // elements of a piece
+  const int maps = maps_of(p.maps), GK = G * maps, D = p.dim, V = p.vdim, KS = key_stride(GK, DS);
   const size_t prw = static_cast<size_t>(p.G) * (maps * D + V);
   const size_t koff = static_cast<size_t>(g0) * maps * D;
   const size_t voff = static_cast<size_t>(p.G) * maps * D + static_cast<size_t>(g0) * V;
-  const bool vec16 = p.pool_dtype == VILA_DT_BF16 && (D & 7) == 0 && (V & 7) == 0;
-  const bool vec32 = p.pool_dtype == VILA_DT_F32 && (D & 3) == 0 && (V & 3) == 0;
+  const int kq = GK * D / E, per = kq + (with_v ? G * V / E : 0), total = BK * per;
+  for (int first = threadIdx.x; first < total; first += kLoads * nthreads) {
+    uint4 u[kLoads];
+    int jj[kLoads], x[kLoads];
+#pragma unroll
+    for (int i = 0; i < kLoads; ++i) {
+      const int item = first + i * nthreads;
+      jj[i] = item / per;
+      x[i] = item - jj[i] * per;
+      u[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (item < total && j0 + jj[i] < nkeys) {
+        const size_t at = pool_row(pt, p.page, j0 + jj[i]) * prw + (x[i] < kq ? koff + x[i] * E : voff + (x[i] - kq) * E);
+        u[i] = BF16 ? __ldg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.pool) + at))
+                    : __ldg(reinterpret_cast<const uint4*>(static_cast<const float*>(p.pool) + at));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kLoads; ++i) {
+      if (first + i * nthreads >= total) break;
+      const int e = x[i] * E, g = e / D;
+      float* d = x[i] < kq ? Ks + jj[i] * KS + g * DS + (e - g * D) : Vs + jj[i] * G * V4 + (x[i] - kq) * E;
+      if (BF16) {
+        *reinterpret_cast<float4*>(d) = make_float4(__uint_as_float(u[i].x << 16), __uint_as_float(u[i].x & 0xffff0000u),
+                                                    __uint_as_float(u[i].y << 16), __uint_as_float(u[i].y & 0xffff0000u));
+        *reinterpret_cast<float4*>(d + 4) = make_float4(__uint_as_float(u[i].z << 16), __uint_as_float(u[i].z & 0xffff0000u),
+                                                        __uint_as_float(u[i].w << 16), __uint_as_float(u[i].w & 0xffff0000u));
+      } else {
+        *reinterpret_cast<uint4*>(d) = u[i];
+      }
+    }
+  }
+}
+
+__device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_paged_attn_params& p,
+                                              const int32_t* pt, int j0, int nkeys, int BK, int D4, int DS, int V4,
+                                              int nwarps, int g0, int G, bool with_v) {
+  const int maps = maps_of(p.maps), GK = G * maps, D = p.dim, V = p.vdim;
+  if (p.pool_dtype == VILA_DT_BF16 && (D & 7) == 0 && (V & 7) == 0) {
+    load_kv_vec<true>(Ks, Vs, p, pt, j0, nkeys, BK, DS, V4, 32 * nwarps, g0, G, with_v);
+    return;
+  }
+  if (p.pool_dtype == VILA_DT_F32 && (D & 3) == 0 && (V & 3) == 0) {
+    load_kv_vec<false>(Ks, Vs, p, pt, j0, nkeys, BK, DS, V4, 32 * nwarps, g0, G, with_v);
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, KS = key_stride(GK, DS);
+  const size_t prw = static_cast<size_t>(p.G) * (maps * D + V);
+  const size_t koff = static_cast<size_t>(g0) * maps * D;
+  const size_t voff = static_cast<size_t>(p.G) * maps * D + static_cast<size_t>(g0) * V;
   for (int jj = warp; jj < BK; jj += nwarps) {
     const int j = j0 + jj;
     float* kd = Ks + jj * KS;
@@ -203,47 +250,14 @@ __device__ __forceinline__ void load_kv_block(float* Ks, float* Vs, const vila_p
       for (int x = lane; x < G * V4; x += 32) vd[x] = 0.f;
       continue;
     }
-    const size_t src = pool_row(pt, p.page, j) * prw;
-    if (vec16) {
-      const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.pool) + src;
-      const uint4* k4 = reinterpret_cast<const uint4*>(base + koff);
-      const uint4* v4 = reinterpret_cast<const uint4*>(base + voff);
-      for (int x = lane; x < (GK * D) >> 3; x += 32) {
-        const uint4 u = __ldg(k4 + x);
-        const int e = x << 3, g = e / D, k = e - g * D;
-        float* d = kd + g * DS + k;
-        *reinterpret_cast<float4*>(d) = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u),
-                                                    __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
-        *reinterpret_cast<float4*>(d + 4) = make_float4(__uint_as_float(u.z << 16), __uint_as_float(u.z & 0xffff0000u),
-                                                        __uint_as_float(u.w << 16), __uint_as_float(u.w & 0xffff0000u));
-      }
-      for (int x = lane; with_v && x < (G * V) >> 3; x += 32) {
-        const uint4 u = __ldg(v4 + x);
-        float* d = vd + (x << 3);
-        *reinterpret_cast<float4*>(d) = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u),
-                                                    __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
-        *reinterpret_cast<float4*>(d + 4) = make_float4(__uint_as_float(u.z << 16), __uint_as_float(u.z & 0xffff0000u),
-                                                        __uint_as_float(u.w << 16), __uint_as_float(u.w & 0xffff0000u));
-      }
-    } else if (vec32) {
-      const float* base = static_cast<const float*>(p.pool) + src;
-      const float4* k4 = reinterpret_cast<const float4*>(base + koff);
-      const float4* v4 = reinterpret_cast<const float4*>(base + voff);
-      for (int x = lane; x < (GK * D) >> 2; x += 32) {
-        const int e = x << 2, g = e / D, k = e - g * D;
-        *reinterpret_cast<float4*>(kd + g * DS + k) = __ldg(k4 + x);
-      }
-      for (int x = lane; with_v && x < (G * V) >> 2; x += 32) *reinterpret_cast<float4*>(vd + (x << 2)) = __ldg(v4 + x);
-    } else {
-      for (int x = lane; x < GK * D4; x += 32) {
-        const int g = x / D4, k = x - g * D4;
-        kd[g * DS + k] = k < D ? ld_any(p.pool, p.pool_dtype, src + koff + static_cast<size_t>(g) * D + k) : 0.f;
-      }
-      const size_t vsrc = src + voff;
-      for (int x = lane; with_v && x < G * V4; x += 32) {
-        const int g = x / V4, k = x - g * V4;
-        vd[x] = k < V ? ld_any(p.pool, p.pool_dtype, vsrc + static_cast<size_t>(g) * V + k) : 0.f;
-      }
+    const size_t src = pool_row(pt, p.page, j) * prw, vsrc = src + voff;
+    for (int x = lane; x < GK * D4; x += 32) {
+      const int g = x / D4, k = x - g * D4;
+      kd[g * DS + k] = k < D ? ld_any(p.pool, p.pool_dtype, src + koff + static_cast<size_t>(g) * D + k) : 0.f;
+    }
+    for (int x = lane; with_v && x < G * V4; x += 32) {
+      const int g = x / V4, k = x - g * V4;
+      vd[x] = k < V ? ld_any(p.pool, p.pool_dtype, vsrc + static_cast<size_t>(g) * V + k) : 0.f;
     }
   }
 }
@@ -267,8 +281,8 @@ __device__ __forceinline__ void combine_maps(const vila_paged_attn_params& p, co
 //   Ss [BQ * H][BK] raw scores | Ps [BQ * H][BK] weights | talk [H * H] | m, l, alpha [BQ * H]
 // H and G count score heads (a head's maps singly), the value heads are GV = G / maps.
 // DS = D4 + 4: consecutive keys start 4 banks apart, so the float4 reads of 8 keys do not collide.
-template <int NACC>
-__global__ void __launch_bounds__(kThreads) paged_attn_kernel(const vila_paged_attn_params p, const AttnShape sh) {
+template <int NACC>   // few accumulators: registers for four CTAs on an SM, whose loads and barriers then overlap
+__global__ void __launch_bounds__(kThreads, NACC <= 2 ? 4 : (NACC <= 8 ? 2 : 1)) paged_attn_kernel(const vila_paged_attn_params p, const AttnShape sh) {
   extern __shared__ __align__(16) float sm[];
   // H, G: the heads this CTA serves (all of them, or one value head with its key and query heads: h0 + h, g0 + g)
   const int maps = maps_of(p.maps), HT = p.H * maps, hs = blockIdx.y % sh.hsplit;

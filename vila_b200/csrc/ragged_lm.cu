@@ -318,63 +318,77 @@ __device__ __forceinline__ void st4_any(void* p, int dt, size_t i, float4 v) {
   *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p) + i) = u;
 }
 
-// A warp takes four outputs at a time (their dot products share the row's loads and overlap); the shared expert's gate,
-// if there is one, is the output after the last.
-template <int TPR, bool VEC>
-__global__ void __launch_bounds__(kRowThreads) moe_route_scores_kernel(const vila_moe_route_params p) {
+// A CTA takes NT tokens; its warps split the outputs, four at a time and for all the tokens (every weight is read once per
+// CTA, the dot products overlap); the shared expert's gate, if there is one, is the output after the last.  Then a warp
+// per token chooses.  A token's sums run in the same order whatever NT is.
+template <int NT, int THREADS, bool VEC>
+__global__ void __launch_bounds__(THREADS) moe_route_scores_kernel(const vila_moe_route_params p) {
   extern __shared__ float z_s[];  // per token: s [experts] | c [experts] | group score [groups]
-  const int wid = threadIdx.x >> 5, lane = lane_id();
-  const int row = row_of<TPR>();
-  if (row >= p.rows) return;
-  const int experts = p.experts, groups = p.groups, keep = p.keep, cols = p.cols;
-  float* s = TPR == 32 ? z_s + wid * (2 * experts + groups) : z_s;
-  float* c = s + experts;
-  float* gs = c + experts;
-  const size_t xb = static_cast<size_t>(row) * p.ldx;
+  const int wid = threadIdx.x >> 5, lane = lane_id(), row0 = blockIdx.x * NT;
+  const int experts = p.experts, groups = p.groups, keep = p.keep, cols = p.cols, per_tok = 2 * experts + groups;
   const int outs = experts + (p.gate_w ? 1 : 0);
-  for (int e0 = 4 * (TPR == 32 ? 0 : wid); e0 < outs; e0 += 4 * (TPR == 32 ? 1 : kRowsPerCta)) {
+  size_t xb[NT];
+#pragma unroll
+  for (int t = 0; t < NT; ++t) xb[t] = static_cast<size_t>(min(row0 + t, p.rows - 1)) * p.ldx;
+  for (int e0 = 4 * wid; e0 < outs; e0 += 4 * (THREADS / 32)) {
     const float* we[4];
-    float a[4] = {0.f, 0.f, 0.f, 0.f};
+    float a[NT][4];
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       const int e = min(e0 + u, outs - 1);
       we[u] = e < experts ? p.w + static_cast<size_t>(e) * cols : p.gate_w;
+#pragma unroll
+      for (int t = 0; t < NT; ++t) a[t][u] = 0.f;
     }
     if (VEC) {
+#pragma unroll 2
       for (int k = 4 * lane; k < cols; k += 128) {
-        const float4 xv = ld4_any(p.x, p.x_dtype, xb + k);
+        float4 wv[4];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const float4 wv = __ldg(reinterpret_cast<const float4*>(we[u] + k));
-          a[u] = fmaf(xv.x, wv.x, a[u]); a[u] = fmaf(xv.y, wv.y, a[u]);
-          a[u] = fmaf(xv.z, wv.z, a[u]); a[u] = fmaf(xv.w, wv.w, a[u]);
+        for (int u = 0; u < 4; ++u) wv[u] = __ldg(reinterpret_cast<const float4*>(we[u] + k));
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+          const float4 xv = ld4_any(p.x, p.x_dtype, xb[t] + k);
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            a[t][u] = fmaf(xv.x, wv[u].x, a[t][u]); a[t][u] = fmaf(xv.y, wv[u].y, a[t][u]);
+            a[t][u] = fmaf(xv.z, wv[u].z, a[t][u]); a[t][u] = fmaf(xv.w, wv[u].w, a[t][u]);
+          }
         }
       }
     } else {
       for (int k = lane; k < cols; k += 32) {
-        const float xv = ld_any(p.x, p.x_dtype, xb + k);
 #pragma unroll
-        for (int u = 0; u < 4; ++u) a[u] = fmaf(xv, we[u][k], a[u]);
+        for (int t = 0; t < NT; ++t) {
+          const float xv = ld_any(p.x, p.x_dtype, xb[t] + k);
+#pragma unroll
+          for (int u = 0; u < 4; ++u) a[t][u] = fmaf(xv, we[u][k], a[t][u]);
+        }
       }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1)
 #pragma unroll
-      for (int u = 0; u < 4; ++u) a[u] += __shfl_xor_sync(0xffffffffu, a[u], o);
+      for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) a[t][u] += __shfl_xor_sync(0xffffffffu, a[t][u], o);
     if (lane == 0) {
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int e = e0 + u;
-        if (e < experts) s[e] = a[u];
-        else if (e < outs) p.gate[row] = sigmoid_f(a[u]);
-      }
+      for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const int e = e0 + u;
+          if (e < experts) z_s[t * per_tok + e] = a[t][u];
+          else if (e < outs && row0 + t < p.rows) p.gate[row0 + t] = sigmoid_f(a[t][u]);
+        }
     }
   }
-  if (TPR == 32) __syncwarp();
-  else {
-    __syncthreads();
-    if (wid != 0) return;
-  }
+  __syncthreads();
+  const int row = row0 + wid;
+  if (wid >= NT || row >= p.rows) return;
+  float* s = z_s + wid * per_tok;
+  float* c = s + experts;
+  float* gs = c + experts;
   float mx = 0.f, inv = 1.f;
   if (p.score == VILA_SCORE_SOFTMAX) {
     mx = -INFINITY;
@@ -883,13 +897,15 @@ int moe_route_scores(const vila_moe_route_params& p, cudaStream_t stream) {
            "moe_route_scores: score=%d group_top=%d", p.score, p.group_top);
   const size_t per_tok = sizeof(float) * (2 * p.experts + p.groups);
   const bool vec = p.cols % 4 == 0 && rows4(p.x, p.ldx, p.x_dtype) && aligned_to(p.w, 16) && (!p.gate_w || aligned_to(p.gate_w, 16));
-#define VB_ROUTE(K, G, S) VB_CUDA(launch_serial(K, dim3(G), dim3(kRowThreads), S, stream, p))
-  if (p.rows <= 1024 || per_tok * kRowsPerCta > 48 * 1024) {   // few tokens, or too many experts for a warp's share
-    if (vec) VB_ROUTE((moe_route_scores_kernel<256, true>), p.rows, per_tok);
-    else VB_ROUTE((moe_route_scores_kernel<256, false>), p.rows, per_tok);
+#define VB_ROUTE(NT, TH, VEC)                                                                                       \
+  VB_CUDA(launch_serial(moe_route_scores_kernel<NT, TH, VEC>, dim3((p.rows + NT - 1) / NT), dim3(TH), NT * per_tok, \
+                        stream, p))
+  if (p.rows <= 256 || 4 * per_tok > 48 * 1024) {   // few tokens (or very many experts): one per CTA of 32 warps
+    if (vec) VB_ROUTE(1, 1024, true);
+    else VB_ROUTE(1, 1024, false);
   } else {
-    if (vec) VB_ROUTE((moe_route_scores_kernel<32, true>), row_grid(p.rows), per_tok * kRowsPerCta);
-    else VB_ROUTE((moe_route_scores_kernel<32, false>), row_grid(p.rows), per_tok * kRowsPerCta);
+    if (vec) VB_ROUTE(4, 256, true);
+    else VB_ROUTE(4, 256, false);
   }
 #undef VB_ROUTE
   return 0;
