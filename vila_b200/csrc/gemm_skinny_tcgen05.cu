@@ -590,8 +590,7 @@ int launch_skinny(const __nv_bfloat16* A, int lda, const __nv_bfloat16* W, int l
   a.ws = ws_ptr ? reinterpret_cast<float*>(static_cast<char*>(ws_ptr) + kCounterBytes) : nullptr;
   a.epi = epi;
   a.dbg = nullptr;
-#ifdef VILA_B200_DEBUG_HOOKS  // profiling aids, compiled OUT of the shipped library (an env var
-                              // must not be able to make a kernel write through an arbitrary pointer)
+#ifdef VILA_B200_DEBUG_HOOKS  // clock stamps, left out of the shipped library: no variable may name a pointer to write to
   if (const char* e = getenv("VILA_B200_GEMM_DEBUG")) {  // hex device pointer (tools/skinny_phase_times.py)
     unsigned long long ptr = 0;
     if (sscanf(e, "%llx", &ptr) == 1) a.dbg = reinterpret_cast<long long*>(ptr);
