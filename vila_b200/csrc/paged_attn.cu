@@ -179,8 +179,8 @@ __device__ __forceinline__ float out_gate(const vila_paged_attn_params& p, int r
 }
 
 // K | V rows of a key block, widened to fp32.  16-byte loads when the head sizes allow (bf16: multiples of 8, fp32:
-// multiples of 4; the pool row is then 16-byte aligned as well): the block's pieces are dealt to all threads, and a thread
-// has kLoads of them in flight before it stores the first.  Otherwise a warp per key, element by element.
+// multiples of 4; the pool row is then 16-byte aligned as well): the block's pieces are dealt to all threads (a warp per
+// key where rows are wide), and a thread has kLoads of them in flight before it stores the first.  Otherwise a warp per key, element by element.
 // g0, G: the value heads g0 .. g0 + G - 1 of the pool row are loaded with their key heads (as many, or one per map).
 constexpr int kLoads = 4;
 
@@ -192,8 +192,41 @@ __device__ __forceinline__ void load_kv_vec(float* Ks, float* Vs, const vila_pag
   const size_t prw = static_cast<size_t>(p.G) * (maps * D + V);
   const size_t koff = static_cast<size_t>(g0) * maps * D;
   const size_t voff = static_cast<size_t>(p.G) * maps * D + static_cast<size_t>(g0) * V;
-  const int kq = GK * D / E, per = kq + (with_v ? G * V / E : 0), total = BK * per;
-  for (int first = threadIdx.x; first < total; first += kLoads * nthreads) {
+  const int kq = GK * D / E, per = kq + (with_v ? G * V / E : 0);   // pieces of a key: k, all
+  auto fetch = [&](size_t row, int x) {
+    const size_t at = row * prw + (x < kq ? koff + x * E : voff + (x - kq) * E);
+    return BF16 ? __ldg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.pool) + at))
+                : __ldg(reinterpret_cast<const uint4*>(static_cast<const float*>(p.pool) + at));
+  };
+  auto store = [&](int jj, int x, uint4 u) {
+    const int e = x * E, g = e / D;
+    float* d = x < kq ? Ks + jj * KS + g * DS + (e - g * D) : Vs + jj * G * V4 + (x - kq) * E;
+    if (BF16) {
+      *reinterpret_cast<float4*>(d) = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u),
+                                                  __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+      *reinterpret_cast<float4*>(d + 4) = make_float4(__uint_as_float(u.z << 16), __uint_as_float(u.z & 0xffff0000u),
+                                                      __uint_as_float(u.w << 16), __uint_as_float(u.w & 0xffff0000u));
+    } else {
+      *reinterpret_cast<uint4*>(d) = u;
+    }
+  };
+  if (per >= 96) {   // wide rows (several heads): a warp per key
+    for (int jj = threadIdx.x >> 5; jj < BK; jj += nthreads >> 5) {
+      const bool ok = j0 + jj < nkeys;
+      const size_t row = ok ? pool_row(pt, p.page, j0 + jj) : 0;
+      for (int first = threadIdx.x & 31; first < per; first += 32 * kLoads) {
+        uint4 u[kLoads];
+#pragma unroll
+        for (int i = 0; i < kLoads; ++i)
+          u[i] = ok && first + 32 * i < per ? fetch(row, first + 32 * i) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+        for (int i = 0; i < kLoads; ++i)
+          if (first + 32 * i < per) store(jj, first + 32 * i, u[i]);
+      }
+    }
+    return;
+  }
+  for (int first = threadIdx.x; first < BK * per; first += kLoads * nthreads) {   // narrow rows: pieces dealt to all threads
     uint4 u[kLoads];
     int jj[kLoads], x[kLoads];
 #pragma unroll
@@ -201,27 +234,11 @@ __device__ __forceinline__ void load_kv_vec(float* Ks, float* Vs, const vila_pag
       const int item = first + i * nthreads;
       jj[i] = item / per;
       x[i] = item - jj[i] * per;
-      u[i] = make_uint4(0u, 0u, 0u, 0u);
-      if (item < total && j0 + jj[i] < nkeys) {
-        const size_t at = pool_row(pt, p.page, j0 + jj[i]) * prw + (x[i] < kq ? koff + x[i] * E : voff + (x[i] - kq) * E);
-        u[i] = BF16 ? __ldg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.pool) + at))
-                    : __ldg(reinterpret_cast<const uint4*>(static_cast<const float*>(p.pool) + at));
-      }
+      u[i] = item < BK * per && j0 + jj[i] < nkeys ? fetch(pool_row(pt, p.page, j0 + jj[i]), x[i]) : make_uint4(0u, 0u, 0u, 0u);
     }
 #pragma unroll
-    for (int i = 0; i < kLoads; ++i) {
-      if (first + i * nthreads >= total) break;
-      const int e = x[i] * E, g = e / D;
-      float* d = x[i] < kq ? Ks + jj[i] * KS + g * DS + (e - g * D) : Vs + jj[i] * G * V4 + (x[i] - kq) * E;
-      if (BF16) {
-        *reinterpret_cast<float4*>(d) = make_float4(__uint_as_float(u[i].x << 16), __uint_as_float(u[i].x & 0xffff0000u),
-                                                    __uint_as_float(u[i].y << 16), __uint_as_float(u[i].y & 0xffff0000u));
-        *reinterpret_cast<float4*>(d + 4) = make_float4(__uint_as_float(u[i].z << 16), __uint_as_float(u[i].z & 0xffff0000u),
-                                                        __uint_as_float(u[i].w << 16), __uint_as_float(u[i].w & 0xffff0000u));
-      } else {
-        *reinterpret_cast<uint4*>(d) = u[i];
-      }
-    }
+    for (int i = 0; i < kLoads; ++i)
+      if (first + i * nthreads < BK * per) store(jj[i], x[i], u[i]);
   }
 }
 
