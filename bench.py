@@ -2290,9 +2290,9 @@ def lightning_lm_block(args, peaks):
         pf = torch.randn(S * top, W, device=dev)
         t = timed_op(lambda: ops.tanh_residual_rows(x, lm.layers[2].norms, out_dtype=bf, a=y1, a_scale=La.ls1, b=y2, b_scale=La.ls2, b_gate=sg,
                                                     part=pf, n_partials=top, idx=idx, weight=wt, experts=E - 4, h=hb, mult=0.5))
-        led["tanh_residual_rows: gated shared + %d routed partials, two norms (2048 rows)" % top] = bytes_(t, S * W * (8 + 2 + 2 + 4 + 4 * top))
+        led["tanh_residual_rows: gated shared + top routed partials, two norms (2048 rows)"] = bytes_(t, S * W * (8 + 2 + 2 + 4 + 4 * top))
         t = timed_op(lambda: ops.residual_norm_rows(x, y1, La.ls1, 1e-5, part=pf, n_partials=top, out_dtype=bf))
-        led["ludazen residual_norm_rows: %d partials, one norm (2048 rows)" % top] = bytes_(t, S * W * (8 + 2 + 2 + 4 * top))
+        led["ludazen residual_norm_rows: top partials, one norm (2048 rows)"] = bytes_(t, S * W * (8 + 2 + 2 + 4 * top))
         # router and experts
         for rows, tag in ((S, "2048 rows"), (B, "decode, 8 rows")):
             by = rows * W * 2 + E * W * 4
